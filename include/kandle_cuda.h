@@ -260,6 +260,8 @@ typedef enum kd_epilogue {
   KD_EPI_NONE = 0,
   KD_EPI_RESIDUAL = 1, /* out = residual + x W^T : `linear` followed by the residual `add`;
                           residual has the output's dtype (bf16, or fp32 residual stream) */
+  KD_EPI_CLAMPED_GLU = 4, /* kd_moe_linear: g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit);
+                             weight rows interleaved like KD_EPI_SWIGLU */
   KD_EPI_SWIGLU = 2    /* out = silu(x Wg^T) * (x Wu^T) : gate/up `linear`, `silu`, `mul`;
                           weight rows interleave 16 gate rows / 16 up rows per 32-row block      */
 } kd_epilogue;
@@ -541,6 +543,63 @@ int kd_allreduce_add_rmsnorm(const kd_tensor* x, const kd_tensor* residual, cons
 int kd_p2p_selftest_silent_peers(int nranks, uint32_t wait_cycles, uint32_t answered_tag);
 int kd_p2p_selftest_dropped_flag(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* norm_out, int drop_rank,
                                  uint32_t wait_cycles);
+
+/* ---------------------------------------------------------------------------------------------
+ * Layers of hybrid decoders (latent attention, gated delta rule, expert feed-forward, Dynamic Tanh).
+ * bf16 (fp32 accumulation; norms, scores, routing, residual, decays and state in fp32) or fp32 throughout,
+ * chosen by the tensors' type.  Positions are a device int32 scalar (graph replay) or a host value.
+ *
+ * kd_linear_ex: out = alpha x W^T (+ residual, fp32 output); x may have any row stride.  With `tail`, out
+ *   has fewer columns than W has rows and the outputs of the remaining rows go to tail in fp32 (a bf16 out
+ *   must then have a multiple of 32 columns to stay on the tensor cores). */
+int kd_linear_ex(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* residual, float alpha, const kd_tensor* out,
+                 const kd_tensor* tail);
+/* x_out[t] = table[ids[t]] * scale (fp32);  h_out = tanh(alpha x_out) * w + b. */
+int kd_embed_dynamic_tanh(const kd_tensor* table, const kd_tensor* ids, float scale, float alpha, const kd_tensor* norm_weight,
+                          const kd_tensor* norm_bias, const kd_tensor* x_out, const kd_tensor* h_out);
+/* x_out = x + sum over splits of mix [splits,T,W] + sum_k weights[t,k] y[slots[t,k]];  h_out = tanh(alpha x_out) * w + b.
+ * mix and y may be NULL; x_out may be x. */
+int kd_residual_dynamic_tanh(const kd_tensor* x, const kd_tensor* mix, const kd_tensor* y, const kd_tensor* slots,
+                             const kd_tensor* weights, float alpha, const kd_tensor* norm_weight, const kd_tensor* norm_bias,
+                             const kd_tensor* x_out, const kd_tensor* h_out);
+/* Router: s = sigmoid(logits [T,E]); the `keep` of `groups` groups with the largest sum of their two largest s stay; the
+ * `top` largest s among them are chosen, weights = s / (their sum + 1e-20).  counts [E] (zero before the call) and
+ * ranks [T,top] number every expert's tokens. */
+int kd_moe_route(const kd_tensor* logits, int top, int groups, int keep, const kd_tensor* ids, const kd_tensor* weights,
+                 const kd_tensor* ranks, const kd_tensor* counts);
+/* Rows of h in expert order: slots[t,k] = offsets[ids[t,k]] + ranks[t,k], x_sorted[slots[t,k]] = h[t]; offsets [E+1]. */
+int kd_moe_gather(const kd_tensor* h, const kd_tensor* ids, const kd_tensor* ranks, const kd_tensor* counts, int experts,
+                  const kd_tensor* slots, const kd_tensor* offsets, const kd_tensor* x_sorted);
+/* out rows of expert e = epilogue(x rows of e * weight[e]^T), weight [E,N,K]; KD_EPI_NONE or KD_EPI_CLAMPED_GLU. */
+int kd_moe_linear(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* offsets, int epilogue, float limit, const kd_tensor* out);
+/* Rotates the queries' last rot_dim dimensions in place (interleaved pairs) and writes the cache row (normed latent,
+ * rotated shared key part) of every token; kv_col < 0: queries only.  proj [B,S,N], cache [B,maxS,width],
+ * cos / sin fp32 [maxS, rot_dim/2]; dense (optional) receives the normed latents as [B*S, kv_rank]. */
+int kd_latent_prep(const kd_tensor* proj, int q_col, int heads, int dim, int rot_dim, int kv_col, int kv_rank,
+                   const kd_tensor* norm_weight, float eps, const kd_tensor* cos, const kd_tensor* sin, const kd_tensor* cache,
+                   const kd_tensor* pos_dev, int pos_host, const kd_tensor* dense);
+/* q_abs [B,S,H,width] = (wuk[h]^T q_unrotated, q_rotated, zeros); wuk [H,dim,kv_rank]. */
+int kd_latent_absorb(const kd_tensor* proj, int q_col, int rot_dim, const kd_tensor* wuk, const kd_tensor* q_abs);
+/* Causal attention of the S queries at position pos on over the cache rows; per row and split the unnormalised sum of
+ * latents, part_o fp32 [B*S*H, splits, kv_rank], and (running maximum in the log2 domain, sum), part_ml [B*S*H, splits, 2]. */
+int kd_latent_attention(const kd_tensor* q_abs, const kd_tensor* cache, int kv_rank, float scale, const kd_tensor* pos_dev,
+                        int pos_host, const kd_tensor* part_o, const kd_tensor* part_ml);
+int kd_latent_attention_splits(int batch, int queries, int heads, int max_seq_len, int* splits_out);
+/* out [T,H*vdim] = wuv_t[h]^T (combined latent sums), wuv_t [H,kv_rank,vdim]; exp(sink[h]) joins the denominator. */
+int kd_latent_values(const kd_tensor* part_o, const kd_tensor* part_ml, const kd_tensor* sink, const kd_tensor* wuv_t,
+                     const kd_tensor* out);
+/* Gated delta rule with a decay per key channel; the projections of proj [B,S,N] pass a causal convolution and silu first.
+ * decay fp32 [T, heads*dim] (before dt_bias), neg_rate = -exp(A_log) [heads], history [B,taps-1,channels] (q, k, v channels
+ * side by side, the inputs before this call), state fp32 [B,heads,rows,cols] as kd_delta_state_shape says, updated in
+ * place; out fp32 [T, heads*vdim].  The history is moved on by kd_delta_out, which divides every head's output by its root
+ * mean square, multiplies by norm_weight [vdim] and sigmoid(gate), and writes proj's type. */
+int kd_delta_rule(const kd_tensor* proj, int q_col, int k_col, int v_col, int b_col, const kd_tensor* decay, int heads, int kv_heads,
+                  int dim, int vdim, const kd_tensor* conv_q, const kd_tensor* conv_k, const kd_tensor* conv_v,
+                  const kd_tensor* neg_rate, const kd_tensor* dt_bias, const kd_tensor* history, const kd_tensor* state,
+                  const kd_tensor* out);
+int kd_delta_state_shape(int dim, int vdim, int* rows_out, int* cols_out);
+int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, float eps, const kd_tensor* proj,
+                 int conv_col, int taps, const kd_tensor* history, const kd_tensor* out);
 
 #ifdef __cplusplus
 }

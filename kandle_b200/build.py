@@ -41,6 +41,8 @@ def build(force: bool = False, verbose: bool = False) -> str:
     sources = sorted(glob.glob(os.path.join(CSRC, "*.cu")))
     headers = sorted(glob.glob(os.path.join(CSRC, "*.cuh"))) + [
         os.path.join(PKG_DIR, "..", "include", "kandle_cuda.h")]
+    if not force and _newer(LIB_PATH, sources + headers):
+        return LIB_PATH       # (also where the object files did not travel with the library)
     objs, jobs = [], []
     for src in sources:
         obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")

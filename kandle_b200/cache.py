@@ -1,0 +1,96 @@
+"""What the layers of a hybrid decoder keep between steps, for a batch of sequences at one position.
+
+  LatentRows   latent attention: one row (normed latent, rotated shared key part) per token,
+               [B, maxS, width]; several layers may read the same rows
+  DeltaState   gated delta rule: the fp32 state matrix of every head and the last inputs of the short
+               convolution; fixed size, carried from token to token
+
+`SequenceCache` owns one such object per layer that has one of its own, the write position shared by
+all layers, and the reset that hands the memory to the next request.
+"""
+from __future__ import annotations
+
+import ctypes
+
+from . import core, lib
+from .core import Tensor
+from .model_utils.pedorax import LatentAttentionSpec
+
+
+def _fill_zero(t: Tensor) -> None:
+    lib.call("kd_fill", ctypes.byref(t._handle.c()), ctypes.c_double(0.0))
+
+
+class LatentRows:
+    """Rows are padded to a multiple of 16 numbers (zeros): whole 32-byte pieces for the bf16 kernels."""
+
+    def __init__(self, spec: LatentAttentionSpec, batch: int, max_seq_len: int, dtype: str):
+        self.width = (spec.kvRank + spec.rotDim + 15) // 16 * 16
+        self.rows = core.zeros((batch, max_seq_len, self.width), dtype)
+
+    def reset(self) -> None:
+        pass                      # rows at and past the write position are never read
+
+    def carried(self) -> list:
+        return []
+
+
+class DeltaState:
+    def __init__(self, spec, batch: int, dtype: str):
+        r, c = ctypes.c_int(0), ctypes.c_int(0)
+        lib.call("kd_delta_state_shape", spec.dim, spec.vdim, ctypes.byref(r), ctypes.byref(c))
+        self.state = core.zeros((batch, spec.heads, r.value, c.value), "float32")
+        self.history = core.zeros((batch, max(spec.taps - 1, 1), spec.channels), dtype)
+
+    def reset(self) -> None:
+        _fill_zero(self.state)
+        _fill_zero(self.history)
+
+    def carried(self) -> list:
+        return [self.state, self.history]
+
+
+class SequenceCache:
+    def __init__(self, layers, batch: int, max_seq_len: int, dtype: str):
+        self.batch, self.max_seq_len = batch, max_seq_len
+        self.pos = 0
+        self._of = []
+        for layer in layers:
+            m = layer.mixer
+            if not isinstance(m, LatentAttentionSpec):
+                self._of.append(DeltaState(m, batch, dtype))
+            elif m.kvFrom is None:
+                self._of.append(LatentRows(m, batch, max_seq_len, dtype))
+            else:
+                self._of.append(self._of[m.kvFrom])
+        self._own = list({id(x): x for x in self._of}.values())
+
+    def of(self, layer: int):
+        return self._of[layer]
+
+    def reset(self) -> None:
+        """Position 0 and zero recurrent state: the sequences are over, new ones may use their place."""
+        for x in self._own:
+            x.reset()
+        self.pos = 0
+
+    def room(self, tokens: int) -> None:
+        if self.pos + tokens > self.max_seq_len:
+            raise ValueError(f"Cache overflow: trying to write to position {self.pos}-{self.pos + tokens}, but maxSeqLen is {self.max_seq_len}")
+
+    def snapshot(self) -> list:
+        """Copies of everything that a step overwrites in place (a cache row can simply be written again)."""
+        return [(t, t.clone()) for x in self._own for t in x.carried()]
+
+    @staticmethod
+    def restore(saved: list) -> None:
+        for t, copy in saved:
+            core.copy_(t, copy)
+            copy.dispose()
+
+    def bytes_per_token(self) -> int:
+        return sum(x.width * (2 if x.rows.dtype == "bfloat16" else 4) for x in self._own if isinstance(x, LatentRows))
+
+    def state_bytes(self) -> int:
+        """Recurrent state per sequence."""
+        return sum(t.numel // self.batch * (2 if t.dtype == "bfloat16" else 4) for x in self._own for t in x.carried())

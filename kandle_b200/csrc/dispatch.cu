@@ -221,3 +221,52 @@ KD_API int kd_qkv_linear_norm_rope_cachewrite(const kd_tensor* x, const kd_tenso
   return gemm_bf16_qkv_rope(px, K, pw, wqkv->strides[0], (int)tokens, (int)K, S, Hq, Hkv, start_pos, eps, (const float*)pc,
                             (const float*)ps, pqw, pkw, pq, pkc, pvc, k_cache->strides[0], k_cache->strides[1], k_cache->strides[2]);
 }
+
+// One linear for the decoders that mix layer types: strided activation rows, a few rows or many, bf16 or
+// fp32, any size, optionally a residual and a block of trailing weight rows whose outputs stay fp32.
+KD_API int kd_linear_ex(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* residual, float alpha, const kd_tensor* out,
+                        const kd_tensor* tail) {
+  KD_TRY(require_init());
+  KD_REQUIRE(x && weight && out, "null tensor");
+  KD_REQUIRE(x->ndim == 2 && x->strides[1] == 1 && weight->ndim == 2 && is_contiguous(weight) && x->dtype == weight->dtype &&
+                 (x->dtype == KD_BF16 || x->dtype == KD_F32) && x->shape[1] == weight->shape[1],
+             "kd_linear_ex needs x [M,K] with unit column stride and a contiguous weight [N,K] of its type");
+  KD_REQUIRE(out->ndim == 2 && out->strides[1] == 1 && out->shape[0] == x->shape[0] && (out->dtype == KD_F32 || out->dtype == x->dtype), "out must be [M,N], fp32 or of x's type");
+  const int64_t M = x->shape[0], K = x->shape[1], N = weight->shape[0], n_out = out->shape[1], ldo = out->strides[0], ldx = x->strides[0];
+  KD_REQUIRE(n_out <= N && (tail != nullptr || n_out == N), "out has %lld columns for %lld weight rows", (long long)n_out, (long long)N);
+  if (tail) KD_REQUIRE(tail->ndim == 2 && tail->dtype == KD_F32 && is_contiguous(tail) && tail->shape[0] == M && tail->shape[1] == N - n_out && n_out < N, "tail must be contiguous fp32 [M, N - out columns]");
+  if (residual) KD_REQUIRE(!tail && out->dtype == KD_F32 && residual->dtype == KD_F32 && residual->ndim == 2 && is_contiguous(residual) && residual->shape[0] == M && residual->shape[1] == N, "residual must be contiguous fp32 [M,N] for an fp32 output");
+  if (M == 0) return KD_OK;
+  void *px, *pw, *po, *pr = nullptr, *pt = nullptr;
+  KD_TRY(tensor_ptr(x, &px));
+  KD_TRY(tensor_ptr(weight, &pw));
+  KD_TRY(tensor_ptr(out, &po));
+  if (residual) KD_TRY(tensor_ptr(residual, &pr));
+  if (tail) KD_TRY(tensor_ptr(tail, &pt));
+  const uintptr_t all = reinterpret_cast<uintptr_t>(px) | reinterpret_cast<uintptr_t>(pw) | reinterpret_cast<uintptr_t>(po) |
+                        reinterpret_cast<uintptr_t>(pr) | reinterpret_cast<uintptr_t>(pt);
+  if (x->dtype == KD_BF16 && (all & 15) == 0 && K % 8 == 0 && N % 8 == 0 && ldx % 8 == 0 && ldo % (out->dtype == KD_F32 ? 4 : 8) == 0 &&
+      (!tail || (n_out % 32 == 0 && (N - n_out) % 4 == 0)) && M < (1ll << 30)) {
+    const bool f32 = out->dtype == KD_F32;
+    // a handful of rows: stream the weights through the swapped kernel (its outputs are dense)
+    if (M <= 64 && !residual && ldo == n_out && !(tail && f32) && (f32 || alpha == 1.0f))
+      return gemm_bf16_skinny(px, ldx, pw, K, (int)M, (int)N, (int)K, 1, f32 ? (float*)po : nullptr, f32 ? nullptr : po, 0, alpha, (float*)pt,
+                              (int)n_out, tail ? (int)tail->shape[1] : 0);
+    if (alpha == 1.0f)
+      return gemm_bf16_bias_act(px, ldx, pw, K, po, ldo, f32, pr, N, (int)M, (int)N, (int)K, residual ? KD_EPI_RESIDUAL : KD_EPI_NONE, nullptr, 0,
+                                (float*)pt, tail ? (int)n_out : 0, tail ? tail->shape[1] : 0);
+  }
+  // exact fp32, and sizes the tensor-core kernels do not take
+  for (int part = 0; part < (tail ? 2 : 1); ++part) {
+    kd_tensor w = *weight;
+    w.shape[0] = part ? N - n_out : n_out;
+    w.offset += part ? n_out * K : 0;
+    kd_matmul_cfg cfg = {};
+    cfg.M = M; cfg.N = w.shape[0]; cfg.K = K;
+    cfg.transpose_b = 1;
+    cfg.alpha = alpha; cfg.beta = 1.0f;
+    cfg.has_c = residual != nullptr;
+    KD_TRY(matmul_f32_dispatch(&cfg, x, &w, residual, part ? tail : out));
+  }
+  return KD_OK;
+}

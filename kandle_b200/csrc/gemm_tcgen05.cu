@@ -106,8 +106,18 @@ struct GemmParams {
   __nv_bfloat16* k_cache;
   __nv_bfloat16* v_cache;
   int64_t kc_b, kc_h, kc_s;
+  // columns from tail_col on (a multiple of 32) go to `tail` in fp32: projections that must not be
+  // rounded (router logits) share the GEMM of the ones that may
+  float* tail;
+  int tail_col;
+  int64_t ld_tail;
+  // grouped: A rows [group_off[g], group_off[g+1]) meet W rows [g N, (g+1) N); offsets in device memory
+  const int* group_off;
+  int groups;
+  float glu_limit;        // epi == 4: clamped GLU, see clamped_glu_f
 };
 
+constexpr int GEMM_MAX_GROUPS = 1024;
 constexpr int GEMM_BM = 128;
 constexpr int GEMM_BK = 64;
 constexpr int GEMM_THREADS = 192;
@@ -138,6 +148,15 @@ __device__ __forceinline__ float silu_f(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
   return x * r;
+}
+
+// g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
+__device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(g * (-1.702f * 1.4426950408889634f)));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return g * r * (u + 1.0f);
 }
 
 template <int BLOCK_N, int STAGES>
@@ -176,9 +195,45 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
+  pdl_wait();      // nothing above touches global memory
+  pdl_trigger();   // after the TMEM allocation (see common.cuh)
 
   const int num_k_blocks = (p.K + GEMM_BK - 1) / GEMM_BK;
-  const int total_tiles = p.num_m_tiles * p.num_n_tiles;
+  int num_m_tiles = p.num_m_tiles;
+  __shared__ int group_tile[GEMM_MAX_GROUPS + 1];      // first 128-row tile of every group
+  if (p.groups > 0) {
+    if (warp == 0) {
+      int carry = 0;
+      for (int base = 0; base < p.groups; base += 32) {
+        const int g = base + lane;
+        const int c = g < p.groups ? (p.group_off[g + 1] - p.group_off[g] + GEMM_BM - 1) / GEMM_BM : 0;
+        int inc = c;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const int v = __shfl_up_sync(0xffffffffu, inc, o);
+          if (lane >= o) inc += v;
+        }
+        if (g < p.groups) group_tile[g] = carry + inc - c;
+        carry += __shfl_sync(0xffffffffu, inc, 31);
+      }
+      if (lane == 0) group_tile[p.groups] = carry;
+    }
+    __syncthreads();
+    num_m_tiles = group_tile[p.groups];
+  }
+  const int total_tiles = num_m_tiles * p.num_n_tiles;
+  // first A row, end of the valid rows and first W row of tile row m_tile
+  auto locate = [&](int m_tile, int& row0, int& row_end, int& w_row) {
+    if (p.groups == 0) { row0 = m_tile * GEMM_BM; row_end = p.M; w_row = 0; return; }
+    int lo = 0, hi = p.groups - 1;                     // last group whose first tile is <= m_tile
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (group_tile[mid] <= m_tile) lo = mid; else hi = mid - 1;
+    }
+    row0 = p.group_off[lo] + (m_tile - group_tile[lo]) * GEMM_BM;
+    row_end = p.group_off[lo + 1];
+    w_row = lo * p.N;
+  };
 
   if (warp == 0) {
     if (lane == 0) {
@@ -187,12 +242,14 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
       bool ok = true;
       for (int tile = blockIdx.x; ok && tile < total_tiles; tile += gridDim.x) {
         const int m_tile = tile / p.num_n_tiles, n_tile = tile - m_tile * p.num_n_tiles;
+        int row0, row_end, w_row;
+        locate(m_tile, row0, row_end, w_row);
         for (int kb = 0; kb < num_k_blocks; ++kb) {
           if (!mbar_wait(&empty[stage], phase ^ 1, abort_flag, p.err, 201)) { ok = false; break; }
           uint8_t* sa = smem + stage * STAGE_BYTES;
           mbar_arrive_expect_tx(&full[stage], STAGE_BYTES);
-          tma_load_2d(sa, &tmap_a, &full[stage], kb * GEMM_BK, m_tile * GEMM_BM);
-          tma_load_2d(sa + A_BYTES, &tmap_b, &full[stage], kb * GEMM_BK, n_tile * BLOCK_N);
+          tma_load_2d(sa, &tmap_a, &full[stage], kb * GEMM_BK, row0);
+          tma_load_2d(sa + A_BYTES, &tmap_b, &full[stage], kb * GEMM_BK, w_row + n_tile * BLOCK_N);
           if (++stage == STAGES) { stage = 0; phase ^= 1; }
         }
       }
@@ -234,12 +291,14 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
     uint32_t acc_phase = 0;
     for (int tile = blockIdx.x; tile < total_tiles; tile += gridDim.x) {
       const int m_tile = tile / p.num_n_tiles, n_tile = tile - m_tile * p.num_n_tiles;
+      int row0, row_end, w_row;
+      locate(m_tile, row0, row_end, w_row);
       bool ok = mbar_wait(&tmem_full[acc], acc_phase, abort_flag, p.err, 204);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const int row = m_tile * GEMM_BM + q * 32 + lane;
-      const bool row_ok = row < p.M;
+      const int row = row0 + q * 32 + lane;
+      const bool row_ok = row < row_end;
       bool released = false;   // accumulator already handed back inside the branch
       const uint32_t t_row = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(acc * BLOCK_N);
       if (BLOCK_N == 256 && p.epi == 3) {
@@ -311,14 +370,20 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                                                             pack_bf16(__uint_as_float(x[g * 8 + 6]), __uint_as_float(x[g * 8 + 7])));
           }
         }
-      } else if (p.epi == 2) {
-        // SiLU(gate) * up.  Weight rows interleave 16 gate rows with the 16 matching up rows, so each
+      } else if (p.epi == 2 || p.epi == 4) {
+        // SiLU(gate) * up, or the clamped GLU.  Weight rows interleave 16 gate rows with the 16 matching up rows, so each
         // 32-column chunk of the accumulator holds 16 (gate, up) pairs and yields 16 outputs.
         __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(p.out) + (int64_t)row * p.ldo + (int64_t)n_tile * (BLOCK_N / 2);
         auto process = [&](uint32_t (&r)[32], const int c0) {
           const int col = n_tile * (BLOCK_N / 2) + c0 / 2;
           if (row_ok && col + 16 <= p.N / 2) {
             uint32_t o[8];
+            if (p.epi == 4) {
+#pragma unroll
+              for (int e = 0; e < 8; ++e)
+                o[e] = pack_bf16(clamped_glu_f(__uint_as_float(r[2 * e]), __uint_as_float(r[16 + 2 * e]), p.glu_limit),
+                                 clamped_glu_f(__uint_as_float(r[2 * e + 1]), __uint_as_float(r[16 + 2 * e + 1]), p.glu_limit));
+            } else
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
               const float a0 = silu_f(__uint_as_float(r[2 * e])) * __uint_as_float(r[16 + 2 * e]);
@@ -359,6 +424,15 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
         auto process = [&](uint32_t (&r)[32], const int c0) {
           if (row_ok) {
             const int col0 = n_tile * BLOCK_N + c0;
+            if (p.tail != nullptr && col0 >= p.tail_col) {
+              float* trow = p.tail + (int64_t)row * p.ld_tail + (col0 - p.tail_col);
+#pragma unroll
+              for (int j = 0; j < 8; ++j)
+                if (col0 + j * 4 + 4 <= p.N)
+                  *reinterpret_cast<float4*>(trow + j * 4) = make_float4(__uint_as_float(r[j * 4]), __uint_as_float(r[j * 4 + 1]),
+                                                                         __uint_as_float(r[j * 4 + 2]), __uint_as_float(r[j * 4 + 3]));
+              return;
+            }
             if (p.bias != nullptr) {
 #pragma unroll
               for (int j = 0; j < 4; ++j) {
@@ -520,11 +594,12 @@ static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, GemmParams&
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM));
     configured[ctx().device & 63] = true;
   }
-  p.num_m_tiles = (p.M + GEMM_BM - 1) / GEMM_BM;
+  // (grouped: every group may end in a partial tile, and groups without rows have none)
+  p.num_m_tiles = (p.M + GEMM_BM - 1) / GEMM_BM + (p.groups ? (p.groups < p.M ? p.groups : p.M) : 0);
   p.num_n_tiles = (p.N + BLOCK_N - 1) / BLOCK_N;
-  const int total = p.num_m_tiles * p.num_n_tiles;
-  const int grid = total < ctx().sm_count ? total : ctx().sm_count;
-  gemm_bf16_tcgen05_kernel<BLOCK_N, STAGES><<<grid, GEMM_THREADS, SMEM, ctx().stream>>>(ta, tb, p);
+  const int64_t total = (int64_t)p.num_m_tiles * p.num_n_tiles;
+  const int grid = total < ctx().sm_count ? (int)total : ctx().sm_count;
+  KD_CUDA_CHECK(launch_ex(gemm_bf16_tcgen05_kernel<BLOCK_N, STAGES>, dim3(grid), dim3(GEMM_THREADS), (size_t)SMEM, ta, tb, p));
   return after_launch("gemm_bf16_tcgen05_kernel");
 }
 
@@ -535,7 +610,8 @@ int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, void* out,
 }
 
 int gemm_bf16_bias_act(const void* A, int64_t lda, const void* W, int64_t ldw, void* out, int64_t ldo, int out_f32,
-                       const void* resid, int64_t ldr, int M, int N, int K, int epi, const void* bias, int act) {
+                       const void* resid, int64_t ldr, int M, int N, int K, int epi, const void* bias, int act, float* tail,
+                       int tail_col, int64_t ld_tail) {
   KD_REQUIRE(M > 0 && N > 0 && K > 0, "gemm: empty problem");
   KD_REQUIRE((bias == nullptr && act == 0) || epi == 0 || epi == 1, "gemm: bias / activation combine only with the plain and residual epilogues");
   KD_REQUIRE((reinterpret_cast<uintptr_t>(bias) & 15) == 0, "gemm: bias must be 16-byte aligned");
@@ -547,8 +623,12 @@ int gemm_bf16_bias_act(const void* A, int64_t lda, const void* W, int64_t ldw, v
     KD_REQUIRE(resid != nullptr && ldr % (out_f32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(resid) & 15) == 0,
                "gemm: residual operand must be 16-byte aligned");
   if (epi == 2) KD_REQUIRE(N % 32 == 0 && !out_f32, "gemm: SwiGLU epilogue needs N %% 32 == 0 and a bf16 output");
+  if (tail != nullptr)
+    KD_REQUIRE(epi == 0 && tail_col % 32 == 0 && tail_col < N && ld_tail % 4 == 0 && (reinterpret_cast<uintptr_t>(tail) & 15) == 0,
+               "gemm: the fp32 tail starts at a multiple of 32 columns (got %d of %d) and is 16-byte aligned", tail_col, N);
   GemmParams p{};
   p.M = M; p.N = N; p.K = K;
+  p.tail = tail; p.tail_col = tail_col; p.ld_tail = ld_tail;
   p.out = out; p.ldo = ldo; p.out_f32 = out_f32;
   p.resid = resid; p.ldr = ldr;
   p.epi = epi;
@@ -569,6 +649,29 @@ int gemm_bf16_bias_act(const void* A, int64_t lda, const void* W, int64_t ldw, v
     return launch_gemm<128, 6>(ta, tb, p);
   }
   KD_TRY(make_tmap_bf16_2d(&tb, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, 64, GEMM_BK));
+  return launch_gemm<64, 8>(ta, tb, p);
+}
+
+// out[rows of g, N or N/2] = epilogue(A[rows of g, K] * W[g][N, K]^T) for all groups g (experts) in one launch.
+int gemm_bf16_grouped(const void* A, const void* W, void* out, const int* group_off, int R, int groups, int N, int K, int glu, float limit) {
+  KD_REQUIRE(R > 0 && groups > 0 && groups <= GEMM_MAX_GROUPS && K % 8 == 0, "grouped gemm: %d rows, %d groups, K=%d", R, groups, K);
+  const int n_out = glu ? N / 2 : N;
+  GemmParams p{};
+  p.M = R; p.N = N; p.K = K;
+  p.out = out; p.ldo = n_out;
+  p.epi = glu ? 4 : 0;
+  p.glu_limit = limit;
+  p.wide_store = n_out % 16 == 0 && (reinterpret_cast<uintptr_t>(out) & 31) == 0;
+  p.group_off = group_off; p.groups = groups;
+  p.err = ctx().error_flag;
+  CUtensorMap ta, tb;
+  KD_TRY(make_tmap_bf16_2d(&ta, A, (uint64_t)R, (uint64_t)K, (uint64_t)K, GEMM_BM, GEMM_BK));
+  // the widest weight tile that still gives every SM a tile
+  const int64_t m_tiles = (R + GEMM_BM - 1) / GEMM_BM + (groups < R ? groups : R) / 2;
+  const int bn = N >= 256 && m_tiles * ((N + 255) / 256) >= ctx().sm_count ? 256 : N > 64 && m_tiles * ((N + 127) / 128) >= ctx().sm_count ? 128 : 64;
+  KD_TRY(make_tmap_bf16_2d(&tb, W, (uint64_t)groups * N, (uint64_t)K, (uint64_t)K, bn, GEMM_BK));
+  if (bn == 256) return launch_gemm<256, 4>(ta, tb, p);
+  if (bn == 128) return launch_gemm<128, 6>(ta, tb, p);
   return launch_gemm<64, 8>(ta, tb, p);
 }
 
@@ -614,8 +717,12 @@ struct SkinnyParams {
   int splits, kblocks_per_split, stages;
   uint32_t tmem_cols;
   float* out_f32;         // [splits][Mb][N]
+  int64_t ldo;            // row stride of out_bf16
   __nv_bfloat16* out_bf16;  // [Mb][N] (or [Mb][N/2] with the SiLU*up epilogue), only with splits == 1
   int swiglu;             // rows of W interleave 16 gate / 16 up rows: write silu(gate)*up
+  float* tail;            // weight rows from tail_row on: fp32 [Mb][ld_tail] instead of the bf16 output
+  int tail_row, ld_tail;
+  float alpha;            // factor of the fp32 outputs
   int* err;
 };
 
@@ -729,8 +836,9 @@ gemm_skinny_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
           for (int i = 0; i < 16; ++i) {
             const int m = c0 + i;
             if (m < p.Mb) {
-              if (p.out_bf16) p.out_bf16[(int64_t)m * p.N + n] = __float2bfloat16_rn(__uint_as_float(r[i]));
-              else p.out_f32[((int64_t)split * p.Mb + m) * p.N + n] = __uint_as_float(r[i]);
+              if (p.tail && n >= p.tail_row) p.tail[(int64_t)m * p.ld_tail + (n - p.tail_row)] = __uint_as_float(r[i]);
+              else if (p.out_bf16) p.out_bf16[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(__uint_as_float(r[i]));
+              else p.out_f32[((int64_t)split * p.Mb + m) * p.N + n] = __uint_as_float(r[i]) * p.alpha;
             }
           }
         }
@@ -761,7 +869,7 @@ int gemm_skinny_auto_splits(int N, int K) {
 // x [Mb<=128, K] bf16, W [N, K] bf16 -> fp32 partials [splits][Mb][N] (or bf16 [Mb][N] when
 // out_bf16 != NULL and splits == 1).
 int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int Mb, int N, int K, int splits,
-                     float* out_f32, void* out_bf16, int swiglu) {
+                     float* out_f32, void* out_bf16, int swiglu, float alpha, float* tail, int tail_row, int ld_tail) {
   KD_REQUIRE(Mb >= 1 && Mb <= 128, "skinny gemm: %d rows; this path handles 1..128", Mb);
   KD_REQUIRE(N > 0 && K > 0 && K % 8 == 0, "skinny gemm: K=%d must be a positive multiple of 8", K);
   KD_REQUIRE(splits >= 1, "skinny gemm: splits must be >= 1");
@@ -790,6 +898,9 @@ int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int
   p.out_f32 = out_f32;
   p.out_bf16 = static_cast<__nv_bfloat16*>(out_bf16);
   p.swiglu = swiglu;
+  p.alpha = alpha;
+  p.tail = tail; p.tail_row = tail_row; p.ld_tail = ld_tail;
+  p.ldo = tail ? tail_row : N;
   p.err = ctx().error_flag;
   CUtensorMap tw, tx;
   KD_TRY(make_tmap_bf16_2d(&tw, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, 128, GEMM_BK));

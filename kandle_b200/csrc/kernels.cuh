@@ -26,7 +26,10 @@ int attention_f32_dispatch(const kd_tensor* q, const kd_tensor* k, const kd_tens
 int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, void* out, int64_t ldo, int out_f32,
               const void* resid, int64_t ldr, int M, int N, int K, int epi);
 int gemm_bf16_bias_act(const void* A, int64_t lda, const void* W, int64_t ldw, void* out, int64_t ldo, int out_f32,
-              const void* resid, int64_t ldr, int M, int N, int K, int epi, const void* bias, int act);
+              const void* resid, int64_t ldr, int M, int N, int K, int epi, const void* bias, int act, float* tail = nullptr,
+              int tail_col = 0, int64_t ld_tail = 0);
+// Grouped form: rows [group_off[g], group_off[g+1]) of A against W[g] [N,K]; glu: clamped GLU over interleaved rows.
+int gemm_bf16_grouped(const void* A, const void* W, void* out, const int* group_off, int R, int groups, int N, int K, int glu, float limit);
 // Tensor-core attention; sets *handled = 1 when it took the call.
 int attention_tc_try(const kd_tensor* q, const kd_tensor* k, const kd_tensor* v, const kd_tensor* out,
                      const AttnParams& p, int* handled);
@@ -37,7 +40,8 @@ int gemm_bf16_qkv_rope(const void* A, int64_t lda, const void* W, int64_t ldw, i
 int gemm_skinny_auto_splits(int N, int K);
 // x [Mb<=128,K] * W[N,K]^T -> fp32 partials [splits][Mb][N], or bf16 [Mb][N] when out_bf16 != NULL (splits == 1).
 int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int Mb, int N, int K, int splits,
-                     float* out_f32, void* out_bf16, int swiglu);
+                     float* out_f32, void* out_bf16, int swiglu, float alpha = 1.0f, float* tail = nullptr, int tail_row = 0,
+                     int ld_tail = 0);
 size_t attention_decode_scratch_bytes(int B, int Hkv, int group, int splits, int D);
 int attention_decode(const kd_tensor* q, const kd_tensor* k, const kd_tensor* v, const kd_tensor* out, float scale,
                      const int* ctx_dev, int ctx_host, const int* block_table, int max_pages, int splits,

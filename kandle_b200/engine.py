@@ -59,7 +59,113 @@ class RandomInit:
         self.seed, self.std = int(seed), float(std)
 
 
-class Qwen3Engine:
+class DecoderEngine:
+    """What the decoder engines share: the generation loop, the sampler, and decode steps captured once
+    as a CUDA graph and replayed.  An engine provides
+
+      prefill(ids)               runs the prompt, returns the next token per sequence (device int64 [B])
+      _decode_state(B)           buffers of a decode step: "ids" [B], "scalars" [write position, context
+                                 length], "graph", "B", ...
+      _enqueue_decode_step(d)    one step for d["ids"] at the device position; leaves the next ids there
+    """
+
+    def _init_decoding(self, max_batch: int, max_seq_len: int) -> None:
+        self.B, self.max_seq_len = max_batch, max_seq_len
+        self._decode = None
+        self.pos = 0
+        self.use_pdl = True
+        self.sampler = None   # None: greedy argmax; else dict(temperature, top_k, top_p, rng), see set_sampler
+
+    def _warm_decode_step(self, d: dict) -> None:
+        """The eager step before a capture (see start_decode)."""
+        self._enqueue_decode_step(d)
+
+    def set_sampler(self, temperature: float = 1.0, top_k: int = 0, top_p: float = 1.0, seed: int = 0) -> None:
+        """Next tokens are drawn on the device (kd_sample: temperature, top-k, top-p, multinomial, the
+        reference's `sample` of packages/model-utils/src/sampling/index.ts:103-238) instead of the
+        greedy argmax.  The uniform numbers come from a seeded host generator, one per sequence and
+        step (128 bytes uploaded per step).  set_sampler(None) restores greedy decoding."""
+        self.dispose()       # a captured decode graph holds the old choice
+        if temperature is None:
+            self.sampler = None
+            return
+        self.sampler = {"temperature": float(temperature), "top_k": int(top_k), "top_p": float(top_p),
+                        "rng": np.random.Generator(np.random.PCG64(seed))}
+
+    def _next_tokens(self, logits2d: Tensor, uniforms, out_ids: Tensor) -> None:
+        if self.sampler is None:
+            lib.call("kd_argmax", _r(logits2d), _r(out_ids))
+        else:
+            sp = self.sampler
+            lib.call("kd_sample", _r(logits2d), ctypes.c_double(sp["temperature"]), sp["top_k"], ctypes.c_double(sp["top_p"]), 1,
+                     _r(uniforms), _r(out_ids), None)
+
+    def _fresh_uniforms(self, t: Tensor) -> None:
+        u = self.sampler["rng"].random(t.shape[0], dtype=np.float32)
+        core._backend().upload(t._handle, u)
+
+    def start_decode(self, first_tokens: Tensor, use_graph: bool = True) -> dict:
+        """Prepares the decode state after a prefill: next input ids = first_tokens (device int64 [B]),
+        write position = prompt length.  With use_graph the step is captured once (after one eager
+        warm-up step on a scratch position) and replayed by decode_step()."""
+        B = first_tokens.shape[0]
+        d = self._decode_state(B)
+        if self.pos + 1 > self.max_seq_len:
+            raise ValueError("Cache overflow: no room left for decode steps")
+        be = core._backend()
+        if use_graph and d["graph"] is None:
+            # warm-up at the current position: sizes the library's scratch and the allocator's caches
+            # (nothing may allocate while capturing); the cache row it writes is overwritten by the
+            # first real step, which runs at the same position.
+            core.copy_(d["ids"], first_tokens)
+            be.upload(d["scalars"]._handle, np.array([self.pos, self.pos + 1], np.int32))
+            self._warm_decode_step(d)
+            lib.call("kd_graph_begin")
+            try:
+                self._enqueue_decode_step(d)
+            finally:
+                g = ctypes.c_uint64(0)
+                lib.call("kd_graph_end", ctypes.byref(g))
+            d["graph"] = g.value
+        core.copy_(d["ids"], first_tokens)
+        be.upload(d["scalars"]._handle, np.array([self.pos, self.pos + 1], np.int32))
+        d["use_graph"] = use_graph
+        return d
+
+    def decode_step(self) -> Tensor:
+        """Runs one step; returns the device int64 [B] tensor holding the tokens just produced."""
+        d = self._decode
+        if self.pos + 1 > self.max_seq_len:
+            raise ValueError(f"Cache overflow: position {self.pos} but maxSeqLen is {self.max_seq_len}")
+        if self.sampler is not None:
+            self._fresh_uniforms(d["uniforms"])     # read by the (replayed) sampling kernel of this step
+        if d["use_graph"]:
+            lib.call("kd_graph_launch", ctypes.c_uint64(d["graph"]))
+        else:
+            self._enqueue_decode_step(d)
+        self.pos += 1
+        return d["ids"]
+
+    def generate(self, ids, steps: int, use_graph: bool = True) -> np.ndarray:
+        """Generation (greedy, or sampled after set_sampler): prefill + `steps` tokens (the first comes from the prefill).  Returns
+        int64 [B, steps] on the host; every step's ids are read back, as the reference does."""
+        tok = self.prefill(ids)
+        B = tok.shape[0]
+        out = np.empty((B, steps), dtype=np.int64)
+        out[:, 0] = tok.dataAsync()
+        if steps > 1:
+            self.start_decode(tok, use_graph)
+            for t in range(1, steps):
+                out[:, t] = self.decode_step().dataAsync()
+        return out
+
+    def dispose(self) -> None:
+        if self._decode is not None and self._decode.get("graph"):
+            lib.call("kd_graph_destroy", ctypes.c_uint64(self._decode["graph"]))
+        self._decode = None
+
+
+class Qwen3Engine(DecoderEngine):
     def __init__(self, cfg: Qwen3Config, weights, max_batch: int, max_seq_len: int, tp_size: int = 1, tp_rank: int = 0,
                  paged: bool = False, page_table: np.ndarray | None = None):
         """weights: HuggingFace-style names -> float32 arrays (rounded to bf16 on upload), or a
@@ -73,7 +179,7 @@ class Qwen3Engine:
         (packages/model-utils/src/kv-cache.ts:164-212), same tokens."""
         self.cfg = cfg
         self.tp = int(tp_size)
-        self.B, self.max_seq_len = max_batch, max_seq_len
+        self._init_decoding(max_batch, max_seq_len)
         c = cfg
         if c.numAttentionHeads % self.tp or c.numKeyValueHeads % self.tp or c.intermediateSize % self.tp:
             raise ValueError(f"heads / intermediate size do not divide over {self.tp} ranks")
@@ -128,9 +234,6 @@ class Qwen3Engine:
             self.v_cache = [core.zeros((self.B, self.Hkv, max_seq_len, self.D), "bfloat16") for _ in range(self.L)]
         self.scale = 1.0 / math.sqrt(self.D)
         self._prefill_bufs = {}
-        self._decode = None
-        self.pos = 0
-        self.use_pdl = True
         self.use_early_kv = os.environ.get("KD_EARLY_KV", "1") != "0"
         # decode: run o_proj .. next layer's QKV as one persistent kernel per layer (kd_decode_layer_chain);
         # tensor parallelism needs an all-reduce after o_proj and down_proj, so it keeps separate kernels
@@ -143,7 +246,6 @@ class Qwen3Engine:
         # tensor parallel decode: sum the partial outputs over ranks through mapped peer memory when
         # the host program has connected the peer buffers (parallel.init_peer_buffers), else NCCL
         self.use_p2p = True
-        self.sampler = None   # None: greedy argmax; else dict(temperature, top_k, top_p, rng), see set_sampler
 
     def _random_weights(self, init: RandomInit, rank: int) -> None:
         c, tp, D = self.cfg, self.tp, self.D
@@ -187,30 +289,6 @@ class Qwen3Engine:
 
     def _norm(self, x, w, out, resid=None, sum_out=None):
         lib.call("kd_add_rmsnorm", _r(x), _r(resid), _r(w), ctypes.c_float(self.cfg.rmsNormEps), _r(sum_out), _r(out))
-
-    def set_sampler(self, temperature: float = 1.0, top_k: int = 0, top_p: float = 1.0, seed: int = 0) -> None:
-        """Next tokens are drawn on the device (kd_sample: temperature, top-k, top-p, multinomial, the
-        reference's `sample` of packages/model-utils/src/sampling/index.ts:103-238) instead of the
-        greedy argmax.  The uniform numbers come from a seeded host generator, one per sequence and
-        step (128 bytes uploaded per step).  set_sampler(None) restores greedy decoding."""
-        self.dispose()       # a captured decode graph holds the old choice
-        if temperature is None:
-            self.sampler = None
-            return
-        self.sampler = {"temperature": float(temperature), "top_k": int(top_k), "top_p": float(top_p),
-                        "rng": np.random.Generator(np.random.PCG64(seed))}
-
-    def _next_tokens(self, logits2d: Tensor, uniforms, out_ids: Tensor) -> None:
-        if self.sampler is None:
-            lib.call("kd_argmax", _r(logits2d), _r(out_ids))
-        else:
-            sp = self.sampler
-            lib.call("kd_sample", _r(logits2d), ctypes.c_double(sp["temperature"]), sp["top_k"], ctypes.c_double(sp["top_p"]), 1,
-                     _r(uniforms), _r(out_ids), None)
-
-    def _fresh_uniforms(self, t: Tensor) -> None:
-        u = self.sampler["rng"].random(t.shape[0], dtype=np.float32)
-        core._backend().upload(t._handle, u)
 
     def _allreduce(self, t) -> None:
         lib.call("kd_allreduce_sum", _r(t))
@@ -471,63 +549,3 @@ class Qwen3Engine:
             t.dispose()
         if table is not None:
             table.dispose()
-
-    def start_decode(self, first_tokens: Tensor, use_graph: bool = True) -> dict:
-        """Prepares the decode state after a prefill: next input ids = first_tokens (device int64 [B]),
-        write position = prompt length.  With use_graph the step is captured once (after one eager
-        warm-up step on a scratch position) and replayed by decode_step()."""
-        B = first_tokens.shape[0]
-        d = self._decode_state(B)
-        if self.pos + 1 > self.max_seq_len:
-            raise ValueError("Cache overflow: no room left for decode steps")
-        be = core._backend()
-        if use_graph and d["graph"] is None:
-            # warm-up at the current position: sizes the library's scratch and the allocator's caches
-            # (nothing may allocate while capturing); the cache row it writes is overwritten by the
-            # first real step, which runs at the same position.
-            core.copy_(d["ids"], first_tokens)
-            be.upload(d["scalars"]._handle, np.array([self.pos, self.pos + 1], np.int32))
-            self._enqueue_decode_step(d)
-            lib.call("kd_graph_begin")
-            try:
-                self._enqueue_decode_step(d)
-            finally:
-                g = ctypes.c_uint64(0)
-                lib.call("kd_graph_end", ctypes.byref(g))
-            d["graph"] = g.value
-        core.copy_(d["ids"], first_tokens)
-        be.upload(d["scalars"]._handle, np.array([self.pos, self.pos + 1], np.int32))
-        d["use_graph"] = use_graph
-        return d
-
-    def decode_step(self) -> Tensor:
-        """Runs one step; returns the device int64 [B] tensor holding the tokens just produced."""
-        d = self._decode
-        if self.pos + 1 > self.max_seq_len:
-            raise ValueError(f"Cache overflow: position {self.pos} but maxSeqLen is {self.max_seq_len}")
-        if self.sampler is not None:
-            self._fresh_uniforms(d["uniforms"])     # read by the (replayed) sampling kernel of this step
-        if d["use_graph"]:
-            lib.call("kd_graph_launch", ctypes.c_uint64(d["graph"]))
-        else:
-            self._enqueue_decode_step(d)
-        self.pos += 1
-        return d["ids"]
-
-    def generate(self, ids, steps: int, use_graph: bool = True) -> np.ndarray:
-        """Generation (greedy, or sampled after set_sampler): prefill + `steps` tokens (the first comes from the prefill).  Returns
-        int64 [B, steps] on the host; every step's ids are read back, as the reference does."""
-        tok = self.prefill(ids)
-        B = tok.shape[0]
-        out = np.empty((B, steps), dtype=np.int64)
-        out[:, 0] = tok.dataAsync()
-        if steps > 1:
-            self.start_decode(tok, use_graph)
-            for t in range(1, steps):
-                out[:, t] = self.decode_step().dataAsync()
-        return out
-
-    def dispose(self) -> None:
-        if self._decode is not None and self._decode.get("graph"):
-            lib.call("kd_graph_destroy", ctypes.c_uint64(self._decode["graph"]))
-        self._decode = None

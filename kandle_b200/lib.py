@@ -178,6 +178,20 @@ _SIGNATURES = {
     "kd_attention_decode": [_T, _T, _T, _T, ctypes.c_int, ctypes.c_float, ctypes.c_int, _T],
     "kd_attention_decode_noalloc": [_T, _T, _T, _T, ctypes.c_int, ctypes.c_float, ctypes.c_int, _T],
     "kd_attention_decode_paged": [_T, _T, _T, _T, _T, ctypes.c_int, ctypes.c_float, ctypes.c_int, _T],
+    "kd_linear_ex": [_T, _T, _T, ctypes.c_float, _T, _T],
+    "kd_embed_dynamic_tanh": [_T, _T, ctypes.c_float, ctypes.c_float, _T, _T, _T, _T],
+    "kd_residual_dynamic_tanh": [_T, _T, _T, _T, _T, ctypes.c_float, _T, _T, _T, _T],
+    "kd_moe_route": [_T, ctypes.c_int, ctypes.c_int, ctypes.c_int, _T, _T, _T, _T],
+    "kd_moe_gather": [_T, _T, _T, _T, ctypes.c_int, _T, _T, _T],
+    "kd_moe_linear": [_T, _T, _T, ctypes.c_int, ctypes.c_float, _T],
+    "kd_latent_prep": [_T] + [ctypes.c_int] * 6 + [_T, ctypes.c_float, _T, _T, _T, _T, ctypes.c_int, _T],
+    "kd_latent_absorb": [_T, ctypes.c_int, ctypes.c_int, _T, _T],
+    "kd_latent_attention": [_T, _T, ctypes.c_int, ctypes.c_float, _T, ctypes.c_int, _T, _T],
+    "kd_latent_attention_splits": [ctypes.c_int] * 4 + [ctypes.POINTER(ctypes.c_int)],
+    "kd_latent_values": [_T, _T, _T, _T, _T],
+    "kd_delta_rule": [_T] + [ctypes.c_int] * 4 + [_T] + [ctypes.c_int] * 4 + [_T] * 8,
+    "kd_delta_state_shape": [ctypes.c_int, ctypes.c_int, ctypes.POINTER(ctypes.c_int), ctypes.POINTER(ctypes.c_int)],
+    "kd_delta_out": [_T, _T, _T, ctypes.c_float, _T, ctypes.c_int, ctypes.c_int, _T, _T],
 }
 
 
