@@ -588,6 +588,10 @@ int kd_latent_attention_splits(int batch, int queries, int heads, int max_seq_le
 /* out [T,H*vdim] = wuv_t[h]^T (combined latent sums), wuv_t [H,kv_rank,vdim]; exp(sink[h]) joins the denominator. */
 int kd_latent_values(const kd_tensor* part_o, const kd_tensor* part_ml, const kd_tensor* sink, const kd_tensor* wuv_t,
                      const kd_tensor* out);
+/* Prompts and portions with keys and values expanded: kv bf16 [B, pos+S, heads*dim | heads*vdim] = latents x [W_uk; W_uv]^T,
+ * the shared rotated key part read from the cache rows; causal from position pos on; sink may be NULL.  tcgen05. */
+int kd_latent_prefill(const kd_tensor* proj, int q_col, int heads, int dim, int rot_dim, const kd_tensor* kv, int vdim,
+                      const kd_tensor* cache, int kv_rank, const kd_tensor* sink, float scale, int pos, const kd_tensor* out);
 /* Gated delta rule with a decay per key channel; the projections of proj [B,S,N] pass a causal convolution and silu first.
  * decay fp32 [T, heads*dim] (before dt_bias), neg_rate = -exp(A_log) [heads], history [B,taps-1,channels] (q, k, v channels
  * side by side, the inputs before this call), state fp32 [B,heads,rows,cols] as kd_delta_state_shape says, updated in

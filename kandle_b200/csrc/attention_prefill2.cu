@@ -28,6 +28,12 @@
 // exponentials on the FMA pipe instead (round-to-nearest split, cubic polynomial, exponent added
 // with integer arithmetic) was measured and made the kernel 7 % slower: more instructions.  Mathematics as in attention_tcgen05.cu / the reference
 // shader (packages/backend-webgpu/src/kernels/attention/builder.ts:138-329).
+//
+// Latent attention (DR > 0) is the same kernel with deeper scores: query and key rows are D unrotated
+// dimensions followed by DR rotated ones, and the rotated key part, which all heads share, comes straight
+// from the cache rows through a tensor map of its own.  With D = 128, DR = 64 both query tiles and two key
+// tiles take 192 KB, so V has one slot instead of two.  Queries may start behind the first key (a portion
+// of a prompt), and a per-head sink may join the softmax denominator.
 #include "common.cuh"
 #include "kernels.cuh"
 #include "sm100.cuh"
@@ -62,6 +68,8 @@ __device__ __forceinline__ void fa2_add2(float& s0, float& s1, float a0, float a
 struct Fa2Params {
   int B, Hq, Hkv, Sq, Skv;
   int causal;
+  int q_off;           // position of query 0 (causal: query i sees keys 0 .. q_off + i)
+  const float* sink;   // [Hq] added to the denominator as exp(sink), or null
   int pair_heads;      // 1: sub-tiles are two heads of one KV group; 0: two consecutive query tiles
   int num_q_tiles;     // 128-row tiles in Sq
   float scale_log2;
@@ -70,15 +78,21 @@ struct Fa2Params {
   int* err;
 };
 
-constexpr int FA2_BQ = 128, FA2_BKV = 128, FA2_THREADS = 384, FA2_NSLOT = 4;
+constexpr int FA2_BQ = 128, FA2_BKV = 128, FA2_THREADS = 384;
 
-template <int D>
+constexpr int FA2_NK = 2;
+constexpr int fa2_nv(int D, int DR) { return D == 128 && DR > 0 ? 1 : 2; }
+
+template <int D, int DR>
 __global__ void __launch_bounds__(FA2_THREADS, 1)
 flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                                const __grid_constant__ CUtensorMap tmap_v, Fa2Params p) {
+                                const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_kr, Fa2Params p) {
   constexpr int SLABS = D / 64;
-  constexpr int Q_BYTES = FA2_BQ * D * 2;
-  constexpr int KV_BYTES = FA2_BKV * D * 2;
+  constexpr int QK_SLABS = (D + DR) / 64;
+  constexpr int NK = FA2_NK, NV = fa2_nv(D, DR);
+  constexpr int Q_BYTES = FA2_BQ * (D + DR) * 2;
+  constexpr int K_BYTES = FA2_BKV * (D + DR) * 2;
+  constexpr int V_BYTES = FA2_BKV * D * 2;
   constexpr int SLAB_BYTES = FA2_BKV * 128;
   constexpr uint32_t TMEM_COLS = 512;
   // TMEM columns: S of sub-tile t at 128 t, O at 256 + D t
@@ -88,10 +102,11 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* q_smem = smem;                                  // [2][Q_BYTES]
-  uint8_t* ring = q_smem + 2 * Q_BYTES;                    // [NSLOT][KV_BYTES]: K0 V0 K1 V1 ...
-  uint64_t* bars = reinterpret_cast<uint64_t*>(ring + FA2_NSLOT * KV_BYTES);
+  uint8_t* k_ring = q_smem + 2 * Q_BYTES;                  // [NK][K_BYTES]
+  uint8_t* v_ring = k_ring + NK * K_BYTES;                 // [NV][V_BYTES]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_ring + NV * V_BYTES);
   uint64_t* q_full = bars;          // 1
-  uint64_t* t_full = bars + 1;      // 4
+  uint64_t* t_full = bars + 1;      // 4: K slots, then V slots
   uint64_t* t_empty = bars + 5;     // 4
   uint64_t* s_full = bars + 9;      // 2 (per sub-tile)
   uint64_t* p_ready = bars + 11;    // 4: [sub-tile][half of the keys]
@@ -117,7 +132,7 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
 #pragma unroll
     for (int t = 0; t < 2; ++t) {
       if (q0[t] >= p.Sq) { nblk[t] = 0; kv_end[t] = 0; continue; }
-      kv_end[t] = p.causal ? min(p.Skv, q0[t] + FA2_BQ) : p.Skv;
+      kv_end[t] = p.causal ? min(p.Skv, p.q_off + q0[t] + FA2_BQ) : p.Skv;
       nblk[t] = (kv_end[t] + FA2_BKV - 1) / FA2_BKV;
     }
   }
@@ -125,7 +140,7 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int s = 0; s < FA2_NSLOT; ++s) { mbar_init(&t_full[s], 1); mbar_init(&t_empty[s], 1); }
+    for (int s = 0; s < NK + NV; ++s) { mbar_init(&t_full[s], 1); mbar_init(&t_empty[s], 1); }
     for (int t = 0; t < 2; ++t) { mbar_init(&s_full[t], 1); mbar_init(&o_done[t], 1); }
     for (int t = 0; t < 4; ++t) mbar_init(&p_ready[t], 4);
     *abort_flag = 0;
@@ -133,6 +148,7 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
     prefetch_tmap(&tmap_q);
     prefetch_tmap(&tmap_k);
     prefetch_tmap(&tmap_v);
+    if (DR > 0) prefetch_tmap(&tmap_kr);
   }
   if (warp == 9) {
     tmem_alloc(tmem_slot, TMEM_COLS);
@@ -151,21 +167,23 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int s = 0; s < SLABS; ++s)
+        for (int s = 0; s < QK_SLABS; ++s)
           tma_load_4d(q_smem + t * Q_BYTES + s * SLAB_BYTES, &tmap_q, q_full, s * 64, q0[t], head[t], b);
       for (int j = 0; j < n_blocks; ++j) {
-        const int tk = 2 * j, tv = 2 * j + 1;
-        const int sk = tk % FA2_NSLOT, sv = tv % FA2_NSLOT;
-        if (!mbar_wait(&t_empty[sk], (uint32_t)(((tk / FA2_NSLOT) & 1) ^ 1), abort_flag, p.err, 401)) break;
-        mbar_arrive_expect_tx(&t_full[sk], KV_BYTES);
+        const int sk = j % NK, sv = j % NV;
+        if (!mbar_wait(&t_empty[sk], (uint32_t)(((j / NK) & 1) ^ 1), abort_flag, p.err, 401)) break;
+        mbar_arrive_expect_tx(&t_full[sk], K_BYTES);
 #pragma unroll
         for (int s = 0; s < SLABS; ++s)
-          tma_load_4d(ring + sk * KV_BYTES + s * SLAB_BYTES, &tmap_k, &t_full[sk], s * 64, j * FA2_BKV, hk, b);
-        if (!mbar_wait(&t_empty[sv], (uint32_t)(((tv / FA2_NSLOT) & 1) ^ 1), abort_flag, p.err, 402)) break;
-        mbar_arrive_expect_tx(&t_full[sv], KV_BYTES);
+          tma_load_4d(k_ring + sk * K_BYTES + s * SLAB_BYTES, &tmap_k, &t_full[sk], s * 64, j * FA2_BKV, hk, b);
+#pragma unroll
+        for (int s = SLABS; s < QK_SLABS; ++s)
+          tma_load_4d(k_ring + sk * K_BYTES + s * SLAB_BYTES, &tmap_kr, &t_full[sk], (s - SLABS) * 64, j * FA2_BKV, 0, b);
+        if (!mbar_wait(&t_empty[NK + sv], (uint32_t)(((j / NV) & 1) ^ 1), abort_flag, p.err, 402)) break;
+        mbar_arrive_expect_tx(&t_full[NK + sv], V_BYTES);
 #pragma unroll
         for (int s = 0; s < SLABS; ++s)
-          tma_load_4d(ring + sv * KV_BYTES + s * SLAB_BYTES, &tmap_v, &t_full[sv], s * 64, j * FA2_BKV, hk, b);
+          tma_load_4d(v_ring + sv * V_BYTES + s * SLAB_BYTES, &tmap_v, &t_full[NK + sv], s * 64, j * FA2_BKV, hk, b);
       }
     }
   } else if (warp == 9) {
@@ -173,14 +191,14 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
       bool ok = mbar_wait(q_full, 0, abort_flag, p.err, 403);
       // S_t(j) = Q_t K(j)^T.  The K tile is waited for once per block (by whichever sub-tile comes first).
       auto issue_qk = [&](int t, int j, bool wait_k) -> bool {
-        const int stage = (2 * j) % FA2_NSLOT;
-        if (wait_k && !mbar_wait(&t_full[stage], (uint32_t)(((2 * j) / FA2_NSLOT) & 1), abort_flag, p.err, 404)) return false;
+        const int stage = j % NK;
+        if (wait_k && !mbar_wait(&t_full[stage], (uint32_t)((j / NK) & 1), abort_flag, p.err, 404)) return false;
         tc_fence_after();
         const uint32_t q_addr = smem_u32(q_smem + t * Q_BYTES);
-        const uint32_t k_addr = smem_u32(ring + stage * KV_BYTES);
+        const uint32_t k_addr = smem_u32(k_ring + stage * K_BYTES);
         const uint32_t d_tmem = tmem_base + (uint32_t)(t * 128);
 #pragma unroll
-        for (int k = 0; k < D / 16; ++k) {
+        for (int k = 0; k < (D + DR) / 16; ++k) {
           const uint32_t off = (uint32_t)((k / 4) * SLAB_BYTES + (k % 4) * 32);
           umma_ss(d_tmem, make_smem_desc_sw128(q_addr + off, 16, 1024), make_smem_desc_sw128(k_addr + off, 16, 1024),
                   IDESC_QK, k != 0 ? 1u : 0u);
@@ -189,11 +207,11 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
         return true;
       };
       // the K slot of block j is released after the last QK^T that reads it
-      auto release_k = [&](int j) { umma_commit(&t_empty[(2 * j) % FA2_NSLOT]); };
+      auto release_k = [&](int j) { umma_commit(&t_empty[j % NK]); };
       auto issue_pv = [&](int t, int j, bool wait_v) -> bool {
-        const int stage = (2 * j + 1) % FA2_NSLOT;
-        if (wait_v && !mbar_wait(&t_full[stage], (uint32_t)(((2 * j + 1) / FA2_NSLOT) & 1), abort_flag, p.err, 406)) return false;
-        const uint32_t v_addr = smem_u32(ring + stage * KV_BYTES);
+        const int stage = j % NV;
+        if (wait_v && !mbar_wait(&t_full[NK + stage], (uint32_t)((j / NV) & 1), abort_flag, p.err, 406)) return false;
+        const uint32_t v_addr = smem_u32(v_ring + stage * V_BYTES);
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           if (!mbar_wait(&p_ready[2 * t + half], (uint32_t)(j & 1), abort_flag, p.err, 405)) return false;
@@ -219,7 +237,7 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
         if (a_now) ok = issue_pv(0, j, true);
         if (ok && a_next) ok = issue_qk(0, j + 1, true);
         if (ok && b_now) ok = issue_pv(1, j, !a_now);
-        if (ok) umma_commit(&t_empty[(2 * j + 1) % FA2_NSLOT]);          // V slot of block j
+        if (ok) umma_commit(&t_empty[NK + j % NV]);          // V slot of block j
         if (ok && b_next) ok = issue_qk(1, j + 1, !a_next);
         if (ok && (a_next || b_next)) release_k(j + 1);
       }
@@ -245,7 +263,7 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
       if (!ok) break;
       tc_fence_after();
       const int kv0 = j * FA2_BKV;
-      const bool masked = (kv0 + FA2_BKV > my_kv_end) || (p.causal && kv0 + FA2_BKV - 1 > my_q0);
+      const bool masked = (kv0 + FA2_BKV > my_kv_end) || (p.causal && kv0 + FA2_BKV - 1 > p.q_off + my_q0);
       // the whole S row of this thread, once
       uint32_t r[128];
 #pragma unroll
@@ -253,7 +271,7 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
       tmem_wait_ld();
       if (masked) {
         // key kv0 + i is visible to this row iff i <= lim
-        const int lim = (p.causal ? min(p.Skv - 1, row) : p.Skv - 1) - kv0;
+        const int lim = (p.causal ? min(p.Skv - 1, p.q_off + row) : p.Skv - 1) - kv0;
 #pragma unroll
         for (int i = 0; i < 128; ++i)
           if (i > lim) r[i] = __float_as_uint(-1e30f);
@@ -322,6 +340,7 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
     }
     if (ok && nb > 0) {
       tc_fence_after();
+      if (p.sink != nullptr) l += exp2f(p.sink[my_head] * 1.4426950408889634f - m_used);
       const float inv_l = 1.0f / l;
       __nv_bfloat16* orow = p.o + (int64_t)b * p.so_b + (int64_t)my_head * p.so_h + (int64_t)row * p.so_s;
 #pragma unroll 1
@@ -356,15 +375,16 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
   }
 }
 
-template <int D>
-static int launch_fa2(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const Fa2Params& p, dim3 grid) {
-  constexpr int SMEM = 2 * FA2_BQ * D * 2 + FA2_NSLOT * FA2_BKV * D * 2 + 1024 + 256;
+template <int D, int DR>
+static int launch_fa2(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tkr, const Fa2Params& p, dim3 grid) {
+  constexpr int SMEM = 2 * FA2_BQ * (D + DR) * 2 + FA2_NK * FA2_BKV * (D + DR) * 2 + fa2_nv(D, DR) * FA2_BKV * D * 2 + 1024 + 256;
+  static_assert(SMEM <= 227 * 1024, "tiles exceed shared memory");
   static bool configured[64] = {false};   // per device: kd_shutdown + kd_init may move the library to another GPU
   if (!configured[ctx().device & 63]) {
-    KD_CUDA_CHECK(cudaFuncSetAttribute(flash_attention_prefill2_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM));
+    KD_CUDA_CHECK(cudaFuncSetAttribute(flash_attention_prefill2_kernel<D, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM));
     configured[ctx().device & 63] = true;
   }
-  flash_attention_prefill2_kernel<D><<<grid, FA2_THREADS, SMEM, ctx().stream>>>(tq, tk, tv, p);
+  flash_attention_prefill2_kernel<D, DR><<<grid, FA2_THREADS, SMEM, ctx().stream>>>(tq, tk, tv, tkr, p);
   return after_launch("flash_attention_prefill2_kernel");
 }
 
@@ -382,8 +402,71 @@ int attention_prefill2(const CUtensorMap& tq, const CUtensorMap& tk, const CUten
   dim3 grid;
   if (p.pair_heads) grid = dim3(p.num_q_tiles, a.Hq / 2, a.B);
   else grid = dim3((p.num_q_tiles + 1) / 2, a.Hq, a.B);
-  if (a.D == 128) return launch_fa2<128>(tq, tk, tv, p, grid);
-  return launch_fa2<64>(tq, tk, tv, p, grid);
+  if (a.D == 128) return launch_fa2<128, 0>(tq, tk, tv, tk, p, grid);
+  return launch_fa2<64, 0>(tq, tk, tv, tk, p, grid);
 }
 
 }  // namespace kd
+
+using namespace kd;
+
+KD_API int kd_latent_prefill(const kd_tensor* proj, int q_col, int heads, int dim, int rot_dim, const kd_tensor* kv, int vdim,
+                             const kd_tensor* cache, int kv_rank, const kd_tensor* sink, float scale, int pos, const kd_tensor* out) {
+  KD_TRY(require_init());
+  KD_REQUIRE(proj && kv && cache && out, "null tensor");
+  KD_REQUIRE((dim == 128 || dim == 64) && rot_dim == 64 && vdim == dim, "kd_latent_prefill handles head sizes 64+64/64 and 128+64/128, got %d+%d/%d", dim, rot_dim, vdim);
+  KD_REQUIRE(proj->ndim == 3 && proj->dtype == KD_BF16 && proj->strides[2] == 1 && proj->strides[0] == proj->strides[1] * proj->shape[1] && proj->strides[1] % 8 == 0,
+             "proj must be bf16 [B,S,N] with evenly spaced, 16-byte aligned rows");
+  const int B = (int)proj->shape[0], S = (int)proj->shape[1], ctx_len = pos + S;
+  KD_REQUIRE(pos >= 0 && q_col >= 0 && q_col % 8 == 0 && q_col + (int64_t)heads * (dim + rot_dim) <= proj->shape[2], "queries exceed the projection row");
+  KD_REQUIRE(kv->ndim == 3 && kv->dtype == KD_BF16 && is_contiguous(kv) && kv->shape[0] == B && kv->shape[1] == ctx_len && kv->shape[2] == (int64_t)heads * (dim + vdim),
+             "kv must be contiguous bf16 [B, pos+S, heads*(dim+vdim)]");
+  KD_REQUIRE(cache->ndim == 3 && cache->dtype == KD_BF16 && cache->strides[2] == 1 && cache->shape[0] >= B && cache->shape[1] >= ctx_len &&
+                 cache->shape[2] >= kv_rank + rot_dim && kv_rank % 8 == 0 && cache->strides[0] % 8 == 0 && cache->strides[1] % 8 == 0,
+             "cache must be bf16 [B,maxS,width] with 16-byte aligned rows and latents");
+  KD_REQUIRE(out->dtype == KD_BF16 && is_contiguous(out) && numel(out) == (int64_t)B * S * heads * vdim, "out must be bf16 [B*S, heads*vdim]");
+  if (B == 0 || S == 0) return KD_OK;
+  Fa2Params p{};
+  if (sink) {
+    KD_REQUIRE(sink->dtype == KD_F32 && is_contiguous(sink) && numel(sink) == heads, "sink must be fp32 [heads]");
+    void* ps;
+    KD_TRY(tensor_ptr(sink, &ps));
+    p.sink = static_cast<const float*>(ps);
+  }
+  void *pp, *pkv, *pc, *po;
+  KD_TRY(tensor_ptr(proj, &pp));
+  KD_TRY(tensor_ptr(kv, &pkv));
+  KD_TRY(tensor_ptr(cache, &pc));
+  KD_TRY(tensor_ptr(out, &po));
+  KD_REQUIRE(((reinterpret_cast<uintptr_t>(pp) | reinterpret_cast<uintptr_t>(pkv) | reinterpret_cast<uintptr_t>(pc) | reinterpret_cast<uintptr_t>(po)) & 15) == 0,
+             "operands must be 16-byte aligned");
+  const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(pp) + q_col;
+  const __nv_bfloat16* k = static_cast<const __nv_bfloat16*>(pkv);
+  const __nv_bfloat16* kr = static_cast<const __nv_bfloat16*>(pc) + kv_rank;
+  const int64_t ld = proj->strides[1], nkv = kv->shape[2];
+  CUtensorMap tq, tk, tv, tkr;
+  {
+    const int64_t ext[4] = {B, heads, S, dim + rot_dim}, st[3] = {ld * S, dim + rot_dim, ld};
+    KD_TRY(make_tmap_bhsd(&tq, q, ext, st, FA2_BQ));
+  }
+  {
+    const int64_t ext[4] = {B, heads, ctx_len, dim}, st[3] = {nkv * ctx_len, dim, nkv};
+    KD_TRY(make_tmap_bhsd(&tk, k, ext, st, FA2_BKV));
+    KD_TRY(make_tmap_bhsd(&tv, k + (int64_t)heads * dim, ext, st, FA2_BKV));
+  }
+  {
+    const int64_t ext[4] = {B, 1, ctx_len, rot_dim}, st[3] = {cache->strides[0], cache->strides[1], cache->strides[1]};
+    KD_TRY(make_tmap_bhsd(&tkr, kr, ext, st, FA2_BKV));
+  }
+  p.B = B; p.Hq = p.Hkv = heads; p.Sq = S; p.Skv = ctx_len;
+  p.causal = 1;
+  p.q_off = pos;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.o = static_cast<__nv_bfloat16*>(po);
+  p.so_b = (int64_t)S * heads * vdim; p.so_h = vdim; p.so_s = (int64_t)heads * vdim;
+  p.num_q_tiles = (S + FA2_BQ - 1) / FA2_BQ;
+  p.err = ctx().error_flag;
+  dim3 grid((p.num_q_tiles + 1) / 2, heads, B);
+  if (dim == 128) return launch_fa2<128, 64>(tq, tk, tv, tkr, p, grid);
+  return launch_fa2<64, 64>(tq, tk, tv, tkr, p, grid);
+}

@@ -52,7 +52,7 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
                                   CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
 // [b, h, s, d] bf16 tensor with element strides st[0..2] (d contiguous); box = [1,1,box_rows,64].
-static int make_tmap_bhsd(CUtensorMap* out, const void* base, const int64_t* ext, const int64_t* st, uint32_t box_rows) {
+int make_tmap_bhsd(CUtensorMap* out, const void* base, const int64_t* ext, const int64_t* st, uint32_t box_rows) {
   static EncodeTiledFn fn = nullptr;
   if (!fn) {
     void* p = nullptr;

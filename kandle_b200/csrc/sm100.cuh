@@ -213,6 +213,8 @@ int make_tmap_bf16_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_
 int make_tmap_bf16_3d(CUtensorMap* out, const void* base, uint64_t d2, uint64_t rows, uint64_t cols, uint64_t stride2,
                       uint64_t row_stride, uint32_t box_rows, uint32_t box_cols);
 
+// [b, h, s, d] (d contiguous; ext = extents, st = strides of b, h, s in elements), box [1, 1, box_rows, 64].
+int make_tmap_bhsd(CUtensorMap* out, const void* base, const int64_t* ext, const int64_t* st, uint32_t box_rows);
 
 // 32-byte global accesses (sm_100: 256-bit vector ld/st).  The address must be 32-byte aligned.
 __device__ __forceinline__ void st_global_v8(void* ptr, const uint32_t (&v)[8]) {

@@ -33,8 +33,6 @@ from .engine import DecoderEngine, RandomInit, _r, interleave_gate_up
 from .model_utils.pedorax import ChannelDeltaSpec, ExpertsSpec, LatentAttentionSpec, PedoraxConfig
 
 KD_EPI_NONE, KD_EPI_CLAMPED_GLU = 0, 4
-# rows per call of the kernels that put tokens on a grid dimension of 65535
-MAX_ABSORB_TOKENS = 1 << 17
 
 
 def _up(n: int, m: int) -> int:
@@ -165,7 +163,7 @@ class _LatentAttention:
         self.sink = Tensor(w.vector(p + "mix.sink", (m.heads,), 0.0), dtype="float32")
         self.wo = w.matrix(p + "mix.o", (eng.W, m.heads * m.vdim))
         self.wukv = None          # [W_uk; W_uv] as stored, for prompts whose keys and values are expanded
-        expandable = eng.dtype == "bfloat16" and m.dim % 64 == 0 and m.rotDim == 64 and m.vdim == 128 and m.dim == 128 and m.kvRank % 8 == 0
+        expandable = eng.dtype == "bfloat16" and m.dim in (64, 128) and m.vdim == m.dim and m.rotDim == 64 and m.kvRank % 8 == 0
         if w.random:
             self.wuk = w.matrix("", (m.heads, m.dim, m.kvRank))
             self.wuv_t = w.matrix("", (m.heads, m.kvRank, m.vdim))
@@ -185,12 +183,13 @@ class _LatentAttention:
         cache = eng.cache.of(self.i).rows
         cache = cache if cache.shape[0] == B else cache.slice([slice(0, B), slice(None), slice(None)])
         expand = self.wukv is not None and pos_dev is None and S >= eng.expand_from
-        dense = ws("latent", (T, m.kvRank), dt) if expand and self.own and B > 1 and pos_host == 0 else None
+        # (the layers that read another layer's rows expand the same dense copy)
+        dense = ws(f"latent{self.i if self.own else m.kvFrom}", (T, m.kvRank), dt) if expand and B > 1 and pos_host == 0 else None
         lib.call("kd_latent_prep", _r(proj3), self.proj.cols["q"], m.heads, m.dim, m.rotDim, self.proj.cols.get("dkv", -1), m.kvRank,
-                 _r(self.norm), ctypes.c_float(eng.cfg.normEps), _r(self.cos), _r(self.sin), _r(cache), _r(pos_dev), pos_host, _r(dense))
+                 _r(self.norm), ctypes.c_float(eng.cfg.normEps), _r(self.cos), _r(self.sin), _r(cache), _r(pos_dev), pos_host, _r(dense) if self.own else None)
         out = ws("mixed", (T, m.heads * m.vdim), dt)
         if expand:
-            eng.expanded_attention(ws, self, proj3, cache, dense, B, S, pos_host, out)
+            self._expanded(eng, ws, proj3, cache, dense, B, S, pos_host, out)
             return out
         width = cache.shape[2]
         splits = ctypes.c_int(0)
@@ -203,6 +202,20 @@ class _LatentAttention:
         lib.call("kd_latent_attention", _r(q_abs), _r(cache), m.kvRank, ctypes.c_float(m.scale), _r(pos_dev), pos_host, _r(part_o), _r(part_ml))
         lib.call("kd_latent_values", _r(part_o), _r(part_ml), _r(self.sink), _r(self.wuv_t), _r(out))
         return out
+
+
+    def _expanded(self, eng: "HybridEngine", ws: _Buffers, proj3: Tensor, cache: Tensor, dense, B: int, S: int, pos: int, out: Tensor) -> None:
+        """Keys and values of the whole context from its latents, then the tcgen05 prefill kernel."""
+        m, ctx = self.m, pos + S
+        n = m.heads * (m.dim + m.vdim)
+        kv = ws("kv", (B, ctx, n), eng.dtype)
+        if dense is not None:
+            eng.linear(dense, self.wukv, kv.view(B * ctx, n))
+        else:
+            for b in range(B):
+                eng.linear(cache.slice([b, slice(0, ctx), slice(0, m.kvRank)]), self.wukv, kv.slice([b, slice(None), slice(None)]))
+        lib.call("kd_latent_prefill", _r(proj3), self.proj.cols["q"], m.heads, m.dim, m.rotDim, _r(kv), m.vdim, _r(cache), m.kvRank,
+                 _r(self.sink), ctypes.c_float(m.scale), pos, _r(out))
 
 
 class _ChannelDelta:
@@ -368,9 +381,10 @@ class HybridEngine(DecoderEngine):
         self.pos = 0
 
     def extend(self, ids, want=None) -> Tensor:
-        """Runs the next tokens ids [B, S] (host int array) of the current sequences.  Returns fp32 logits
+        """Runs the next tokens ids [B, S] (host int array, or a device int32 Tensor) of the current sequences.  Returns fp32 logits
         [B * len(want), V] at the places `want` of the portion, sequence by sequence (default: the last)."""
-        ids = np.ascontiguousarray(ids, dtype=np.int32)
+        if not isinstance(ids, Tensor):
+            ids = np.ascontiguousarray(ids, dtype=np.int32)
         B, S = ids.shape
         if B > self.B:
             raise ValueError(f"{B} sequences exceed the engine's {self.B}")
@@ -382,10 +396,13 @@ class HybridEngine(DecoderEngine):
             raise ValueError(f"places {want} outside a portion of {S} tokens")
         self.cur_B = B
         if S == 1 and self.pos:
-            logits = self._decode_given(ids)
+            logits = self._decode_given(ids.dataAsync() if isinstance(ids, Tensor) else ids)
             return logits if want == [0] else self._take(logits, [b for b in range(B) for _ in want])
-        t = self._prompt("ids", (B * S,), "int32")
-        core._backend().upload(t._handle, ids.reshape(-1))
+        if isinstance(ids, Tensor):
+            t = ids.view(B * S)
+        else:
+            t = self._prompt("ids", (B * S,), "int32")
+            core._backend().upload(t._handle, ids.reshape(-1))
         h = self._run(self._prompt, t, B, S, None, self.pos)
         self.pos += S
         self.cache.pos = self.pos
@@ -402,10 +419,12 @@ class HybridEngine(DecoderEngine):
         return out
 
     def prefill(self, ids, all_logits: bool = False, portion: int | None = None):
-        """New sequences with prompts ids [B, S] (host array), in portions of `portion` tokens (default: whole).
+        """New sequences with prompts ids [B, S] (host array or device int32 Tensor), in portions of `portion` tokens (default: whole).
         Returns the next token per sequence, device int64 [B] (and fp32 logits [B, S, V] with all_logits)."""
-        ids = ids.dataAsync() if isinstance(ids, Tensor) else ids
-        ids = np.ascontiguousarray(ids, dtype=np.int32)
+        if isinstance(ids, Tensor) and portion:
+            ids = ids.dataAsync()
+        if not isinstance(ids, Tensor):
+            ids = np.ascontiguousarray(ids, dtype=np.int32)
         B, S = ids.shape
         self.reset()
         self.cache.room(S)
@@ -413,7 +432,7 @@ class HybridEngine(DecoderEngine):
         for a in range(0, S, step):
             n = min(step, S - a)
             last = a + n == S
-            lg = self.extend(ids[:, a:a + n], list(range(n)) if all_logits else ([n - 1] if last else []))
+            lg = self.extend(ids if n == S else ids[:, a:a + n], list(range(n)) if all_logits else ([n - 1] if last else []))
             if all_logits:
                 parts.append(lg.dataAsync().reshape(B, n, self.V))
         if all_logits:

@@ -189,6 +189,7 @@ _SIGNATURES = {
     "kd_latent_attention": [_T, _T, ctypes.c_int, ctypes.c_float, _T, ctypes.c_int, _T, _T],
     "kd_latent_attention_splits": [ctypes.c_int] * 4 + [ctypes.POINTER(ctypes.c_int)],
     "kd_latent_values": [_T, _T, _T, _T, _T],
+    "kd_latent_prefill": [_T] + [ctypes.c_int] * 4 + [_T, ctypes.c_int, _T, ctypes.c_int, _T, ctypes.c_float, ctypes.c_int, _T],
     "kd_delta_rule": [_T] + [ctypes.c_int] * 4 + [_T] + [ctypes.c_int] * 4 + [_T] * 8,
     "kd_delta_state_shape": [ctypes.c_int, ctypes.c_int, ctypes.POINTER(ctypes.c_int), ctypes.POINTER(ctypes.c_int)],
     "kd_delta_out": [_T, _T, _T, ctypes.c_float, _T, ctypes.c_int, ctypes.c_int, _T, _T],
