@@ -10,26 +10,30 @@
 // triangular solve per chunk and per-channel decays inside every product.  Counted in instructions
 // that is no cheaper than the recurrence itself when the state lives in registers and the arithmetic
 // is packed (fma.rn.f32x2: two per lane and instruction).  And the result does not depend on where a
-// prompt is cut: every token is computed alone, in order, bit for bit the same in any portion.
+// prompt is cut beyond the rounding of the decay products.
 //
 // Mapping.  A state column (one value channel) never meets another one, so a warp owns 32 / LPC
-// groups of 4 columns, and the LPC lanes of a group share its dim rows (32 rows a lane, in quads
-// i LPC + j): 128 state registers a lane whatever the size.  Per token a lane reads its 32 entries of
-// g, k (twice) and q as broadcast 16-byte shared-memory loads, does 4 packed operations per pair of
-// state entries, and the group's S^T k is a butterfly over LPC lanes.
-// A CTA is eight consumer warps (one or more heads) and four helper warps.  The helpers prepare the
+// groups of 8 columns, and the LPC lanes of a group share its dim rows (16 rows a lane, in quads
+// i LPC + j): 128 state registers a lane whatever the size.  Decays are not applied token by token:
+// inside a group of four tokens the state is kept divided by the product P of the decays so far, and
+// the token's vectors carry the factor (k P and q P to read, k / P to write), so a token costs three
+// packed operations per pair of state entries and the group one more.  Where a decay is so small that
+// 1 / P could leave the range of fp32 (below 1e-6), it is applied to the state at that token instead.
+// S^T k is summed over a group's LPC lanes so that every lane ends with its share of the columns; a
+// token's output is summed while the next token's S^T k is, to share the latency.
+// A CTA is eight consumer warps (one or more heads) and eight helper warps.  The helpers prepare the
 // next block of tokens (convolution, silu, unit norms, decays, step sizes) in shared memory while the
 // consumers walk through the current one.
-// Bound: fp32 pipe in prefill (4 dim vdim packed operations / 2 per head and token), HBM in decode
+// Bound: fp32 pipe in prefill (3.25 dim vdim multiply-adds per head and token), HBM in decode
 // (the state is read and written once per token: 8 dim vdim bytes per head and sequence).
 #include "common.cuh"
 #include "kernels.cuh"
 
 namespace kd {
 
-constexpr int DR_CONSUMERS = 8, DR_HELPERS = 4;
+constexpr int DR_CONSUMERS = 8, DR_HELPERS = 8;
 constexpr int DR_THREADS = (DR_CONSUMERS + DR_HELPERS) * 32;
-constexpr int DR_TB = 8;           // tokens per block
+constexpr int DR_TB = 16;          // tokens per block
 constexpr int DR_MAX_TAPS = 8;
 
 struct DeltaParams {
@@ -42,6 +46,7 @@ struct DeltaParams {
   int64_t ld;                      // projection row stride (elements)
   int64_t ld_a;                    // row stride of the decay logits
   float q_scale;
+  int vec_q, vec_v, vec_a;         // rows allow four-channel vector loads (q and k, v, decay logits)
   const float* a;                  // [T, H*dim] decay logits (before dt_bias)
   const float* conv_q;             // [Hk*dim, taps]
   const float* conv_k;
@@ -51,6 +56,10 @@ struct DeltaParams {
   float* state;
   float* o;                        // [T, H*vdim]
 };
+
+// Shared-memory floats of one head and stage: q, k (read and write side), direct decays [TB][dk], decays left at
+// the end of every four tokens [TB/4][dk], v [TB][dv], step sizes and flags [TB].
+__host__ __device__ constexpr int delta_unit_floats(int dk, int dv) { return DR_TB * (4 * dk + dv) + (DR_TB / 4) * dk + 2 * DR_TB; }
 
 template <typename T> __device__ __forceinline__ float dr_f(T v);
 template <> __device__ __forceinline__ float dr_f<float>(float v) { return v; }
@@ -70,128 +79,323 @@ __device__ __forceinline__ float2 mul2(float2 a, float2 b) {
   return d;
 }
 
-// Rounded projections enter through bf16 (FAST: special-function-unit forms, error at fp32 rounding
-// level for these arguments); the fp32 mode uses the accurate library functions.
+// In bf16 mode (FAST) the elementary functions are the special-function unit's, accurate to a few fp32
+// roundings for these arguments; the fp32 mode uses the accurate library functions.
+__device__ __forceinline__ float ex2f(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcpf(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float DR_LOG2E = 1.4426950408889634f;
 template <bool FAST> __device__ __forceinline__ float dr_sigmoid(float x) {
-  return FAST ? __fdividef(1.0f, 1.0f + __expf(-x)) : 1.0f / (1.0f + expf(-x));
+  return FAST ? rcpf(1.0f + ex2f(-DR_LOG2E * x)) : 1.0f / (1.0f + expf(-x));
 }
-template <bool FAST> __device__ __forceinline__ float dr_softplus(float x) {
-  return FAST ? fmaxf(x, 0.f) + __logf(1.0f + __expf(-fabsf(x))) : fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+// exp(rate softplus(x))
+template <bool FAST> __device__ __forceinline__ float dr_decay(float rate, float x) {
+  if (FAST) {
+    const float z = DR_LOG2E * x;
+    return ex2f(rate * (fmaxf(z, 0.f) + __log2f(1.0f + ex2f(-fabsf(z)))));
+  }
+  return expf(rate * (fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)))));
 }
-template <bool FAST> __device__ __forceinline__ float dr_exp(float x) { return FAST ? __expf(x) : expf(x); }
 
-// out[t][i] = silu(causal convolution) of tokens t0 .. t0 + n - 1 (n <= DR_TB), channels i < nc; zeros up to
-// `pad`.  hist holds the taps - 1 inputs before token 0 of this call, [taps-1][C] for the sequence.  A lane
-// keeps the inputs of a channel in registers (four taps, the usual size) or re-reads them (other sizes).
+// Four consecutive channels of a row as they lie in memory.
+template <typename T> struct Raw4;
+template <> struct Raw4<__nv_bfloat16> {
+  uint2 u;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { u = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ void get(float (&v)[4]) const {
+    v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+    v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+  }
+};
+template <> struct Raw4<float> {
+  float4 f;
+  __device__ __forceinline__ void load(const float* p) { f = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ void get(float (&v)[4]) const { v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+};
+
+// The inputs of one short convolution at four tokens: where they are and how to read them.
+template <typename T>
+struct ConvSource {
+  const T* row0;        // token 0 of the sequence, first channel
+  const T* hist;        // the taps - 1 inputs before it
+  int64_t ld, hist_ld;
+  const float* w;       // [nc, taps]
+  int taps, t, S, nc;   // tokens t .. t + 3, those below S
+  bool vec;             // vector loads possible, at most four taps
+};
+
+// Vector form, first half: seven rows of inputs at channels c .. c + 3, no branch between the loads.
+template <typename T>
+__device__ __forceinline__ void conv_fetch(const ConvSource<T>& cs, int c, Raw4<T> (&raw)[7]) {
+  const int halo = cs.taps - 1, cc = c < cs.nc ? c : 0;
+  if (cs.t >= halo && cs.t - halo + 6 < cs.S) {      // all seven rows are rows of this call
+    const T* src = cs.row0 + (cs.t - halo) * cs.ld + cc;
+#pragma unroll
+    for (int r = 0; r < 7; ++r) raw[r].load(src + r * (int)cs.ld);
+    return;
+  }
+#pragma unroll
+  for (int r = 0; r < 7; ++r) {
+    const int tt = cs.t - halo + r;
+    const bool use = r < 3 + cs.taps && tt < cs.S;
+    const T* src = !use ? cs.row0 : tt >= 0 ? cs.row0 + (int64_t)tt * cs.ld : cs.hist + (tt + halo) * cs.hist_ld;
+    raw[r].load(src + cc);
+  }
+}
+
+// Vector form, second half: y[token][channel] = silu(conv), zero for channels past nc and tokens past S.
 template <typename T, bool FAST>
-__device__ __forceinline__ void conv_block(const T* __restrict__ proj, int64_t ld, int64_t row0, int t0, int n, int col, const T* __restrict__ hist,
-                                           int64_t hist_ld, const float* __restrict__ taps_w, int taps, int nc, int pad, float* __restrict__ out,
-                                           int out_ld, int lane) {
-  const int halo = taps - 1;
-  auto input = [&](int t, int i) -> float {
-    return t >= 0 ? dr_f<T>(proj[(row0 + t) * ld + col + i]) : dr_f<T>(hist[(int64_t)(t + halo) * hist_ld + i]);
-  };
-#pragma unroll 1
-  for (int i = lane; i < nc; i += 32) {
-    if (taps == 4) {
-      float x[DR_TB + 3];
+__device__ __forceinline__ void conv_finish(const ConvSource<T>& cs, int c, const Raw4<T> (&raw)[7], float (&y)[4][4]) {
+  float acc[4][4];
 #pragma unroll
-      for (int r = 0; r < DR_TB + 3; ++r) x[r] = r < n + 3 ? input(t0 + r - 3, i) : 0.f;
-      const float w0 = taps_w[i * 4], w1 = taps_w[i * 4 + 1], w2 = taps_w[i * 4 + 2], w3 = taps_w[i * 4 + 3];
+  for (int q = 0; q < 4; ++q)
 #pragma unroll
-      for (int t = 0; t < DR_TB; ++t) {
-        if (t < n) {
-          const float y = fmaf(x[t + 3], w3, fmaf(x[t + 2], w2, fmaf(x[t + 1], w1, x[t] * w0)));
-          out[t * out_ld + i] = y * dr_sigmoid<FAST>(y);
-        }
-      }
-    } else {
-      for (int t = 0; t < n; ++t) {
-        float y = 0.f;
-        for (int j = 0; j < taps; ++j) y = fmaf(input(t0 + t - halo + j, i), taps_w[(int64_t)i * taps + j], y);
-        out[t * out_ld + i] = y * dr_sigmoid<FAST>(y);
+    for (int e = 0; e < 4; ++e) acc[q][e] = 0.f;
+  const int cc = c < cs.nc ? c : 0;
+  float w[4][4];        // [channel][tap]
+  if (cs.taps == 4) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float4 f = __ldg(reinterpret_cast<const float4*>(cs.w) + cc + e);
+      w[e][0] = f.x; w[e][1] = f.y; w[e][2] = f.z; w[e][3] = f.w;
+    }
+  } else {
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) w[e][k] = k < cs.taps ? __ldg(cs.w + (cc + e) * cs.taps + k) : 0.f;
+  }
+#pragma unroll
+  for (int r = 0; r < 7; ++r) {
+    float x[4];
+    raw[r].get(x);
+    // (rows that no token of this call uses meet a zero weight, or a token past S, whose result is dropped)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int k = r - q;
+      if (k >= 0 && k < 4) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[q][e] = fmaf(x[e], w[e][k], acc[q][e]);
       }
     }
   }
-#pragma unroll 1
-  for (int i = nc + lane; i < pad; i += 32)
-    for (int t = 0; t < n; ++t) out[t * out_ld + i] = 0.f;
+#pragma unroll
+  for (int q = 0; q < 4; ++q)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[q][e] = c < cs.nc && cs.t + q < cs.S ? acc[q][e] * dr_sigmoid<FAST>(acc[q][e]) : 0.f;
 }
 
-// x[t] <- scale x[t] / sqrt(sum x[t]^2 + 1e-6) over nc channels; a lane touches the channels it wrote itself.
-__device__ __forceinline__ void unit_rows(float* x, int ld, int n, int nc, float scale, int lane) {
-  for (int t = 0; t < n; ++t) {
-    float ss = 0.f;
-#pragma unroll 1
-    for (int i = lane; i < nc; i += 32) ss = fmaf(x[t * ld + i], x[t * ld + i], ss);
-    ss = warp_sum(ss);
-    const float inv = scale / sqrtf(ss + 1e-6f);
-    for (int i = lane; i < nc; i += 32) x[t * ld + i] *= inv;
-  }
+// Element by element, for sizes or strides that allow no vector loads and for more taps.
+template <typename T, bool FAST>
+__device__ __forceinline__ void conv_slow(const ConvSource<T>& cs, int c, float (&y)[4][4]) {
+  const int halo = cs.taps - 1;
+  for (int q = 0; q < 4; ++q)
+    for (int e = 0; e < 4; ++e) {
+      float acc = 0.f;
+      if (c + e < cs.nc && cs.t + q < cs.S)
+        for (int k = 0; k < cs.taps; ++k) {
+          const int tt = cs.t + q - halo + k;
+          acc = fmaf(dr_f<T>(tt >= 0 ? cs.row0[tt * cs.ld + c + e] : cs.hist[(tt + halo) * cs.hist_ld + c + e]), cs.w[(int64_t)(c + e) * cs.taps + k], acc);
+        }
+      y[q][e] = acc * dr_sigmoid<FAST>(acc);
+    }
 }
+
+// scale / |y[q]| over the warp's channels (CH passes of 128).
+template <bool FAST, int CH>
+__device__ __forceinline__ void unit_scale(const float (&y)[CH][4][4], float scale, float (&inv)[4]) {
+  float ss[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < CH; ++i)
+#pragma unroll
+    for (int q = 0; q < 4; ++q)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss[q] = fmaf(y[i][q][e], y[i][q][e], ss[q]);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) ss[q] += __shfl_xor_sync(0xffffffffu, ss[q], o);
+#pragma unroll
+  for (int q = 0; q < 4; ++q) inv[q] = FAST ? scale * rsqrtf(ss[q] + 1e-6f) : scale / sqrtf(ss[q] + 1e-6f);
+}
+
+// Decays below this are applied to the state at once; products of four larger ones keep 1 / P in range.
+constexpr float DR_SMALL_DECAY = 1e-6f;
 
 template <typename T, int LPC>
 __global__ void __launch_bounds__(DR_THREADS, 1)
 delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_t hist_b, int64_t hist_ld, DeltaParams p) {
   constexpr bool FAST = sizeof(T) == 2;
-  constexpr int DK = 32 * LPC;                 // padded key channels
-  constexpr int CPW = 4 * (32 / LPC);          // value columns per warp
+  constexpr int DK = 16 * LPC;                 // padded key channels
+  constexpr int CH = DK > 128 ? DK / 128 : 1;  // helper passes over the key channels
+  constexpr int CPW = 8 * (32 / LPC);          // value columns per warp
   extern __shared__ __align__(16) float sm[];
   const int dvc = p.wpc * CPW;                 // value columns of a head in this CTA
-  const int unit_floats = DR_TB * (3 * DK + dvc) + DR_TB;
-  // shared memory: [2 stages][upc units]{ q, k, g [TB][DK], v [TB][dvc], beta [TB] }
+  const int unit_floats = delta_unit_floats(DK, dvc);
+  // shared memory: [2 stages][upc units]{ q, kr, kw, d [TB][DK], post [TB/4][DK], v [TB][dvc], (beta, flag) [TB] }
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int units = p.B * p.H;
   const int unit0 = blockIdx.x * p.upc;
   const int col_tile = blockIdx.y * dvc;       // first value column of this CTA inside its heads
-  pdl_wait();
-  pdl_trigger();
   const int n_blk = (p.S + DR_TB - 1) / DR_TB;
 
-  // ---- helper: everything token block `blk` needs, into stage `st`
+  // ---- helper: everything token block `blk` needs, into stage `st`; an item is four tokens of one head
   const int hw = warp - DR_CONSUMERS;
   auto prepare = [&](int blk, int st) {
-    const int t0 = blk * DR_TB, n = min(DR_TB, p.S - t0);
-    for (int item = hw; item < p.upc * 4; item += DR_HELPERS) {
-      const int u = item >> 2, what = item & 3;
-      const int unit = unit0 + u;
-      if (unit >= units) continue;
+    for (int item = hw; item < p.upc * (DR_TB / 4); item += DR_HELPERS) {
+      const int u = item / (DR_TB / 4), grp = item % (DR_TB / 4);
+      const int unit = unit0 + u, t = blk * DR_TB + grp * 4;
+      if (unit >= units || t >= p.S) continue;
       const int b = unit / p.H, h = unit - b * p.H;
       const int hk = h / (p.H / p.Hk);
-      const int64_t row0 = (int64_t)b * p.S;
-      float* base = sm + (st * p.upc + u) * unit_floats;
+      const T* seq = proj + (int64_t)b * p.S * p.ld;
       const T* hb = hist + (int64_t)b * hist_b;
       const int kc = p.Hk * p.dim;             // history channels: q, k, v side by side
-      if (what == 0) {
-        conv_block<T, FAST>(proj, p.ld, row0, t0, n, p.q_col + hk * p.dim, hb + hk * p.dim, hist_ld, p.conv_q + (int64_t)hk * p.dim * p.taps, p.taps,
-                            p.dim, DK, base, DK, lane);
-        unit_rows(base, DK, n, p.dim, p.q_scale, lane);
-      } else if (what == 1) {
-        float* k = base + DR_TB * DK;
-        conv_block<T, FAST>(proj, p.ld, row0, t0, n, p.k_col + hk * p.dim, hb + kc + hk * p.dim, hist_ld, p.conv_k + (int64_t)hk * p.dim * p.taps, p.taps,
-                            p.dim, DK, k, DK, lane);
-        unit_rows(k, DK, n, p.dim, 1.0f, lane);
-      } else if (what == 2) {
-        float* g = base + 2 * DR_TB * DK;
-        const float rate = p.neg_rate[h];
-#pragma unroll 1
-        for (int i = lane; i < DK; i += 32) {
-          if (i < p.dim) {
-            const float bias = p.dt_bias[h * p.dim + i];
-#pragma unroll 4
-            for (int t = 0; t < n; ++t)
-              g[t * DK + i] = dr_exp<FAST>(rate * dr_softplus<FAST>(p.a[(row0 + t0 + t) * p.ld_a + h * p.dim + i] + bias));
+      float* base = sm + (st * p.upc + u) * unit_floats;
+      const ConvSource<T> cq{seq + p.q_col + hk * p.dim, hb + hk * p.dim, p.ld, hist_ld, p.conv_q + (int64_t)hk * p.dim * p.taps, p.taps, t, p.S, p.dim, p.vec_q != 0};
+      const ConvSource<T> ck{seq + p.k_col + hk * p.dim, hb + kc + hk * p.dim, p.ld, hist_ld, p.conv_k + (int64_t)hk * p.dim * p.taps, p.taps, t, p.S, p.dim, p.vec_q != 0};
+      const int at = h * p.vdim + col_tile;
+      const ConvSource<T> cv{seq + p.v_col + at, hb + 2 * kc + at, p.ld, hist_ld, p.conv_v + (int64_t)at * p.taps, p.taps, t, p.S,
+                             max(0, min(dvc, p.vdim - col_tile)), p.vec_v != 0};
+      const int c0 = lane * 4;
+      Raw4<T> raw[7];
+      float g[CH][4][4];
+      const float* a = p.a + ((int64_t)b * p.S + t) * p.ld_a + h * p.dim;
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        const int c = i * 128 + c0;
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const float* ar = a + (t + q < p.S ? q : 0) * p.ld_a;
+          if (p.vec_a) {
+            const float4 f = *reinterpret_cast<const float4*>(ar + (c < p.dim ? c : 0));
+            g[i][q][0] = f.x; g[i][q][1] = f.y; g[i][q][2] = f.z; g[i][q][3] = f.w;
           } else {
-            for (int t = 0; t < n; ++t) g[t * DK + i] = 0.f;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) g[i][q][e] = c + e < p.dim ? ar[c + e] : 0.f;
           }
         }
+      }
+      if (CH == 1 && ck.vec) conv_fetch<T>(ck, c0, raw);
+      // decays
+      const float rate = p.neg_rate[h];
+      float least = 1.f;
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        const int c = i * 128 + c0;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const bool in = c + e < p.dim;
+          const float bias = in ? __ldg(p.dt_bias + h * p.dim + c + e) : 0.f;
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            g[i][q][e] = in && t + q < p.S ? dr_decay<FAST>(rate, g[i][q][e] + bias) : 1.f;
+            least = fminf(least, g[i][q][e]);
+          }
+        }
+      }
+      // running products of the decays since the last one that was applied directly (or the group's start);
+      // g becomes that product, d holds what to multiply the state with where a token is flagged
+      bool flag[4] = {false, false, false, false};
+      if (__any_sync(0xffffffffu, least < DR_SMALL_DECAY)) {
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          bool small = false;
+#pragma unroll
+          for (int i = 0; i < CH; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) small |= g[i][q][e] < DR_SMALL_DECAY;
+          flag[q] = __any_sync(0xffffffffu, small);
+        }
+      }
+      float* dd = base + (3 * DR_TB + grp * 4) * DK;
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        const int c = i * 128 + c0;
+        float P[4] = {1.f, 1.f, 1.f, 1.f};
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) P[e] *= g[i][q][e];
+          if (flag[q]) {
+            if (c < DK) *reinterpret_cast<float4*>(dd + q * DK + c) = make_float4(P[0], P[1], P[2], P[3]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) P[e] = 1.f;
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) g[i][q][e] = P[e];
+        }
+        if (c < DK) *reinterpret_cast<float4*>(base + (4 * DR_TB + grp) * DK + c) = make_float4(P[0], P[1], P[2], P[3]);
+      }
+      float y[CH][4][4], inv[4];
+      // k: read side k P, write side k / P
+      if (CH == 1 && ck.vec) {
+        conv_finish<T, FAST>(ck, c0, raw, y[0]);
+        conv_fetch<T>(cq, c0, raw);
       } else {
-        float* v = base + 3 * DR_TB * DK;
-        const int nc = max(0, min(dvc, p.vdim - col_tile));
-        conv_block<T, FAST>(proj, p.ld, row0, t0, n, p.v_col + h * p.vdim + col_tile, hb + 2 * kc + h * p.vdim + col_tile, hist_ld,
-                            p.conv_v + ((int64_t)h * p.vdim + col_tile) * p.taps, p.taps, nc, dvc, v, dvc, lane);
-        if (lane < n) v[DR_TB * dvc + lane] = dr_sigmoid<FAST>(dr_f<T>(proj[(row0 + t0 + lane) * p.ld + p.b_col + h]));
+        for (int i = 0; i < CH; ++i) conv_slow<T, FAST>(ck, i * 128 + c0, y[i]);
+      }
+      unit_scale<FAST, CH>(y, 1.0f, inv);
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        const int c = i * 128 + c0;
+        if (c < DK) {
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            float kk[4], r[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              kk[e] = y[i][q][e] * inv[q];
+              r[e] = FAST ? rcpf(g[i][q][e]) : 1.0f / g[i][q][e];
+            }
+            *reinterpret_cast<float4*>(base + (DR_TB + grp * 4 + q) * DK + c) =
+                make_float4(kk[0] * g[i][q][0], kk[1] * g[i][q][1], kk[2] * g[i][q][2], kk[3] * g[i][q][3]);
+            *reinterpret_cast<float4*>(base + (2 * DR_TB + grp * 4 + q) * DK + c) = make_float4(kk[0] * r[0], kk[1] * r[1], kk[2] * r[2], kk[3] * r[3]);
+          }
+        }
+      }
+      if (CH == 1 && cq.vec) {
+        conv_finish<T, FAST>(cq, c0, raw, y[0]);
+      } else {
+        for (int i = 0; i < CH; ++i) conv_slow<T, FAST>(cq, i * 128 + c0, y[i]);
+      }
+      if (cv.vec && cv.nc > 0) conv_fetch<T>(cv, c0, raw);
+      unit_scale<FAST, CH>(y, p.q_scale, inv);
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        const int c = i * 128 + c0;
+        if (c < DK) {
+#pragma unroll
+          for (int q = 0; q < 4; ++q)
+            *reinterpret_cast<float4*>(base + (grp * 4 + q) * DK + c) =
+                make_float4(y[i][q][0] * inv[q] * g[i][q][0], y[i][q][1] * inv[q] * g[i][q][1], y[i][q][2] * inv[q] * g[i][q][2],
+                            y[i][q][3] * inv[q] * g[i][q][3]);
+        }
+      }
+      float* v = base + (4 * DR_TB + DR_TB / 4) * DK;
+#pragma unroll 1
+      for (int c = c0; c < dvc; c += 128) {
+        if (cv.vec && cv.nc > 0) {
+          if (c != c0) conv_fetch<T>(cv, c, raw);
+          conv_finish<T, FAST>(cv, c, raw, y[0]);
+        } else {
+          conv_slow<T, FAST>(cv, c, y[0]);
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) *reinterpret_cast<float4*>(v + (grp * 4 + q) * dvc + c) = make_float4(y[0][q][0], y[0][q][1], y[0][q][2], y[0][q][3]);
+      }
+      if (lane < 4) {
+        float* beta = v + DR_TB * dvc;
+        beta[2 * (grp * 4 + lane)] = t + lane < p.S ? dr_sigmoid<FAST>(dr_f<T>(seq[(int64_t)(t + lane) * p.ld + p.b_col + h])) : 0.f;
+        beta[2 * (grp * 4 + lane) + 1] = (lane == 0 ? flag[0] : lane == 1 ? flag[1] : lane == 2 ? flag[2] : flag[3]) ? 1.f : 0.f;
       }
     }
   };
@@ -199,7 +403,9 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
   auto block_barrier = [] { asm volatile("bar.sync 1, %0;" ::"n"(DR_THREADS) : "memory"); };
 
   if (warp >= DR_CONSUMERS) {
-    asm volatile("setmaxnreg.dec.sync.aligned.u32 88;");
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 80;");
+    pdl_wait();
+    pdl_trigger();
     for (int blk = 0; blk < n_blk; ++blk) {
       prepare(blk, blk & 1);      // (its stage was last read two blocks ago, before the previous barrier)
       block_barrier();
@@ -207,101 +413,165 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
     block_barrier();
     return;
   }
-  asm volatile("setmaxnreg.inc.sync.aligned.u32 208;");
-  // ---- consumer state: rows (i LPC + j) 4 + e (i < 8, e < 4) of columns col .. col + 3
+  asm volatile("setmaxnreg.inc.sync.aligned.u32 176;");
+  // ---- consumer state: rows (i LPC + j) 4 + e (i < 4, e < 4) of columns col .. col + 7
+  constexpr int OWN = LPC < 8 ? 8 / LPC : 1;   // columns a lane owns after a sum over its group ...
   const int j = lane % LPC, cg = lane / LPC;
+  const int own = j * 8 / LPC;                 // ... starting here
   const int u = warp / p.wpc, uw = warp - u * p.wpc;
   const int unit = unit0 + u;
-  const int lcol = uw * CPW + cg * 4;          // column inside the CTA's tile
+  const int lcol = uw * CPW + cg * 8;          // column inside the CTA's tile
   const int col = col_tile + lcol;
-  const bool active = u < p.upc && unit < units && col < p.dv_pad;
-  float2 s[4][16];                             // [column][row pair]
+  const bool live = u < p.upc && unit < units;
+  const bool active = live && col < p.dv_pad;
+  float2 s[8][8];                              // [column][row pair]
   float* srow = nullptr;
+#pragma unroll
+  for (int c = 0; c < 8; ++c)
+#pragma unroll
+    for (int r = 0; r < 8; ++r) s[c][r] = make_float2(0.f, 0.f);
+  // (the state was last written a whole step ago, before the launch that the grid-dependency wait is for)
   if (active) {
     srow = p.state + ((int64_t)unit * p.dk_pad + j * 4) * p.dv_pad + col;
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float4 v = *reinterpret_cast<const float4*>(srow + (int64_t)(i * LPC * 4 + e) * p.dv_pad);
-        if (e & 1) { s[0][i * 2 + (e >> 1)].y = v.x; s[1][i * 2 + (e >> 1)].y = v.y; s[2][i * 2 + (e >> 1)].y = v.z; s[3][i * 2 + (e >> 1)].y = v.w; }
-        else { s[0][i * 2 + (e >> 1)].x = v.x; s[1][i * 2 + (e >> 1)].x = v.y; s[2][i * 2 + (e >> 1)].x = v.z; s[3][i * 2 + (e >> 1)].x = v.w; }
-      }
+      for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int w = 0; w < 2; ++w) {
+          const float4 v = *reinterpret_cast<const float4*>(srow + (int64_t)(i * LPC * 4 + e) * p.dv_pad + w * 4);
+          const float vv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            if (e & 1) s[w * 4 + c][i * 2 + (e >> 1)].y = vv[c];
+            else s[w * 4 + c][i * 2 + (e >> 1)].x = vv[c];
+          }
+        }
   }
+  pdl_wait();
+  pdl_trigger();
   block_barrier();
 
-  const int b = active ? unit / p.H : 0, h = active ? unit - b * p.H : 0;
+  auto scale_state = [&](const float4* d4) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float4 d = d4[i * LPC];
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {
+        s[c][2 * i] = mul2(s[c][2 * i], make_float2(d.x, d.y));
+        s[c][2 * i + 1] = mul2(s[c][2 * i + 1], make_float2(d.z, d.w));
+      }
+    }
+  };
+  // Sums x and y over the group's lanes; lane j ends with columns own .. own + OWN - 1 in [0, OWN).
+  auto group_sums = [&](float (&x)[8], float (&y)[8]) {
+    int n = 8;
+#pragma unroll
+    for (int m = LPC / 2; m > 0; m >>= 1) {
+      if (n > 1) {
+        n >>= 1;
+        const bool up = j & m;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (i < n) {
+            const float sx = up ? x[i] : x[i + n], kx = up ? x[i + n] : x[i];
+            const float sy = up ? y[i] : y[i + n], ky = up ? y[i + n] : y[i];
+            x[i] = kx + __shfl_xor_sync(0xffffffffu, sx, m);
+            y[i] = ky + __shfl_xor_sync(0xffffffffu, sy, m);
+          }
+      } else {
+        x[0] += __shfl_xor_sync(0xffffffffu, x[0], m);
+        y[0] += __shfl_xor_sync(0xffffffffu, y[0], m);
+      }
+    }
+  };
+  const int b = live ? unit / p.H : 0, h = live ? unit - b * p.H : 0;
+  float po[8];                                 // this lane's share of the previous token's output
+#pragma unroll
+  for (int c = 0; c < 8; ++c) po[c] = 0.f;
+  const int64_t o_ld = (int64_t)p.H * p.vdim;
+  float* orow = p.o + (int64_t)b * p.S * o_ld + (int64_t)h * p.vdim + col + own;
+  auto store_out = [&](float* ot, bool any) {
+#pragma unroll
+    for (int i = 0; i < OWN; ++i)
+      if (any && (LPC <= 8 || (j & (LPC / 8 - 1)) == 0) && col + own + i < p.vdim) ot[i] = po[i];
+  };
   for (int blk = 0; blk < n_blk; ++blk) {
-    if (active) {
+    // (all lanes of a warp belong to one head; lanes past its columns take part in the shuffles)
+    if (live) {
       const float* base = sm + ((blk & 1) * p.upc + u) * unit_floats;
+      const float* vb = base + (4 * DR_TB + DR_TB / 4) * DK;
       const int t0 = blk * DR_TB, n = min(DR_TB, p.S - t0);
-      float* orow = p.o + ((int64_t)b * p.S + t0) * p.H * p.vdim + (int64_t)h * p.vdim + col;
+#pragma unroll 1
       for (int t = 0; t < n; ++t) {
         const float4* q4 = reinterpret_cast<const float4*>(base + t * DK) + j;
-        const float4* k4 = reinterpret_cast<const float4*>(base + (DR_TB + t) * DK) + j;
-        const float4* g4 = reinterpret_cast<const float4*>(base + (2 * DR_TB + t) * DK) + j;
-        const float4 v4 = *reinterpret_cast<const float4*>(base + 3 * DR_TB * DK + t * dvc + lcol);
-        const float beta = base[3 * DR_TB * DK + DR_TB * dvc + t];
-        float2 acc[4][2];
+        const float4* kr4 = reinterpret_cast<const float4*>(base + (DR_TB + t) * DK) + j;
+        const float4* kw4 = reinterpret_cast<const float4*>(base + (2 * DR_TB + t) * DK) + j;
+        const float2 bf = *reinterpret_cast<const float2*>(vb + DR_TB * dvc + 2 * t);     // step size, flag
+        float v[OWN];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) acc[c][0] = acc[c][1] = make_float2(0.f, 0.f);
+        for (int i = 0; i < OWN; ++i) v[i] = vb[t * dvc + lcol + own + i];
+        if (bf.y != 0.f) scale_state(reinterpret_cast<const float4*>(base + (3 * DR_TB + t) * DK) + j);
+        float2 acc[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const float4 g = g4[i * LPC], k = k4[i * LPC];
+        for (int c = 0; c < 8; ++c) acc[c] = make_float2(0.f, 0.f);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            s[c][2 * i] = mul2(s[c][2 * i], make_float2(g.x, g.y));
-            s[c][2 * i + 1] = mul2(s[c][2 * i + 1], make_float2(g.z, g.w));
-            acc[c][0] = fma2(s[c][2 * i], make_float2(k.x, k.y), acc[c][0]);
-            acc[c][1] = fma2(s[c][2 * i + 1], make_float2(k.z, k.w), acc[c][1]);
-          }
+        for (int i = 0; i < 4; ++i) {
+          const float4 k = kr4[i * LPC];
+#pragma unroll
+          for (int c = 0; c < 8; ++c) acc[c] = fma2(s[c][2 * i], make_float2(k.x, k.y), acc[c]);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) acc[c] = fma2(s[c][2 * i + 1], make_float2(k.z, k.w), acc[c]);
         }
-        float pr[4];
+        float pr[8];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) pr[c] = (acc[c][0].x + acc[c][0].y) + (acc[c][1].x + acc[c][1].y);
+        for (int c = 0; c < 8; ++c) pr[c] = acc[c].x + acc[c].y;
+        // the previous token's output leaves here: its shuffles fill the wait for this token's
+        group_sums(pr, po);
+        store_out(orow + (int64_t)(t0 + t - 1) * o_ld, t0 + t > 0);
 #pragma unroll
-        for (int o = LPC / 2; o > 0; o >>= 1)
+        for (int i = 0; i < OWN; ++i) pr[i] = bf.x * (v[i] - pr[i]);
+        float uu[8];
 #pragma unroll
-          for (int c = 0; c < 4; ++c) pr[c] += __shfl_xor_sync(0xffffffffu, pr[c], o);
-        const float uu[4] = {beta * (v4.x - pr[0]), beta * (v4.y - pr[1]), beta * (v4.z - pr[2]), beta * (v4.w - pr[3])};
+        for (int c = 0; c < 8; ++c) uu[c] = __shfl_sync(0xffffffffu, pr[c % OWN], cg * LPC + c * LPC / 8);
 #pragma unroll
-        for (int c = 0; c < 4; ++c) acc[c][0] = acc[c][1] = make_float2(0.f, 0.f);
+        for (int c = 0; c < 8; ++c) acc[c] = make_float2(0.f, 0.f);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const float4 k = k4[i * LPC], q = q4[i * LPC];
+        for (int i = 0; i < 4; ++i) {
+          const float4 k = kw4[i * LPC], q = q4[i * LPC];
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            const float2 uc = make_float2(uu[c], uu[c]);
-            s[c][2 * i] = fma2(make_float2(k.x, k.y), uc, s[c][2 * i]);
-            s[c][2 * i + 1] = fma2(make_float2(k.z, k.w), uc, s[c][2 * i + 1]);
-            acc[c][0] = fma2(s[c][2 * i], make_float2(q.x, q.y), acc[c][0]);
-            acc[c][1] = fma2(s[c][2 * i + 1], make_float2(q.z, q.w), acc[c][1]);
-          }
+          for (int c = 0; c < 8; ++c) s[c][2 * i] = fma2(make_float2(k.x, k.y), make_float2(uu[c], uu[c]), s[c][2 * i]);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) s[c][2 * i + 1] = fma2(make_float2(k.z, k.w), make_float2(uu[c], uu[c]), s[c][2 * i + 1]);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) acc[c] = fma2(s[c][2 * i], make_float2(q.x, q.y), acc[c]);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) acc[c] = fma2(s[c][2 * i + 1], make_float2(q.z, q.w), acc[c]);
         }
 #pragma unroll
-        for (int c = 0; c < 4; ++c) pr[c] = (acc[c][0].x + acc[c][0].y) + (acc[c][1].x + acc[c][1].y);
-#pragma unroll
-        for (int o = LPC / 2; o > 0; o >>= 1)
-#pragma unroll
-          for (int c = 0; c < 4; ++c) pr[c] += __shfl_xor_sync(0xffffffffu, pr[c], o);
-        // the lanes of a group share the store: lane j writes columns j, j + LPC, ...
-        float* ot = orow + (int64_t)t * p.H * p.vdim;
-#pragma unroll
-        for (int c = 0; c < 4; ++c)
-          if (c % LPC == j % (LPC < 4 ? LPC : 4) && j < 4 && col + c < p.vdim) ot[c] = pr[c];
+        for (int c = 0; c < 8; ++c) po[c] = acc[c].x + acc[c].y;
+        if ((t & 3) == 3 || t + 1 == n) scale_state(reinterpret_cast<const float4*>(base + (4 * DR_TB + (t >> 2)) * DK) + j);
+      }
+      if (blk + 1 == n_blk) {
+        float none[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        group_sums(po, none);
+        store_out(orow + (int64_t)(p.S - 1) * o_ld, true);
       }
     }
     block_barrier();
   }
   if (active) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = i * 2 + (e >> 1);
-        const float4 v = (e & 1) ? make_float4(s[0][r].y, s[1][r].y, s[2][r].y, s[3][r].y) : make_float4(s[0][r].x, s[1][r].x, s[2][r].x, s[3][r].x);
-        *reinterpret_cast<float4*>(srow + (int64_t)(i * LPC * 4 + e) * p.dv_pad) = v;
-      }
+      for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int w = 0; w < 2; ++w) {
+          const int r = i * 2 + (e >> 1);
+          const float4 v = (e & 1) ? make_float4(s[w * 4][r].y, s[w * 4 + 1][r].y, s[w * 4 + 2][r].y, s[w * 4 + 3][r].y)
+                                   : make_float4(s[w * 4][r].x, s[w * 4 + 1][r].x, s[w * 4 + 2][r].x, s[w * 4 + 3][r].x);
+          *reinterpret_cast<float4*>(srow + (int64_t)(i * LPC * 4 + e) * p.dv_pad + w * 4) = v;
+        }
   }
 }
 
@@ -363,7 +633,7 @@ static int f32_vec(const kd_tensor* t, int64_t n, const char* what, const float*
 
 template <typename T, int LPC>
 static int launch_delta(const void* proj, const void* hist, int64_t hist_b, int64_t hist_ld, DeltaParams p) {
-  constexpr int CPW = 4 * (32 / LPC), DK = 32 * LPC;
+  constexpr int CPW = 8 * (32 / LPC), DK = 16 * LPC;
   const int units = p.B * p.H;
   p.wpu = (p.vdim + CPW - 1) / CPW;
   // enough heads to fill the GPU: whole heads per CTA, several if they fit; otherwise split columns
@@ -375,7 +645,7 @@ static int launch_delta(const void* proj, const void* hist, int64_t hist_b, int6
   p.upc = 1;
   while ((p.upc + 1) * p.wpc <= DR_CONSUMERS && units * col_tiles > sms * p.upc) ++p.upc;
   const int dvc = p.wpc * CPW;
-  auto smem_of = [&](int upc) { return 2 * upc * (DR_TB * (3 * DK + dvc) + DR_TB) * 4; };
+  auto smem_of = [&](int upc) { return 2 * upc * delta_unit_floats(DK, dvc) * 4; };
   while (p.upc > 1 && smem_of(p.upc) > 220 * 1024) --p.upc;
   const int smem = smem_of(p.upc);
   KD_REQUIRE(smem <= 227 * 1024, "delta rule: %d x %d heads need too much shared memory", p.dim, p.vdim);
@@ -391,10 +661,10 @@ static int launch_delta(const void* proj, const void* hist, int64_t hist_b, int6
 
 template <typename T>
 static int launch_delta_lpc(const void* proj, const void* hist, int64_t hist_b, int64_t hist_ld, const DeltaParams& p) {
-  if (p.dk_pad == 32) return launch_delta<T, 1>(proj, hist, hist_b, hist_ld, p);
-  if (p.dk_pad == 64) return launch_delta<T, 2>(proj, hist, hist_b, hist_ld, p);
-  if (p.dk_pad == 128) return launch_delta<T, 4>(proj, hist, hist_b, hist_ld, p);
-  return launch_delta<T, 8>(proj, hist, hist_b, hist_ld, p);
+  if (p.dk_pad == 32) return launch_delta<T, 2>(proj, hist, hist_b, hist_ld, p);
+  if (p.dk_pad == 64) return launch_delta<T, 4>(proj, hist, hist_b, hist_ld, p);
+  if (p.dk_pad == 128) return launch_delta<T, 8>(proj, hist, hist_b, hist_ld, p);
+  return launch_delta<T, 16>(proj, hist, hist_b, hist_ld, p);
 }
 
 }  // namespace kd
@@ -407,7 +677,7 @@ KD_API int kd_delta_state_shape(int dim, int vdim, int* rows_out, int* cols_out)
   int r = 32;
   while (r < dim) r *= 2;
   *rows_out = r;
-  *cols_out = (vdim + 3) / 4 * 4;
+  *cols_out = (vdim + 7) / 8 * 8;
   return KD_OK;
 }
 
@@ -444,6 +714,7 @@ KD_API int kd_delta_rule(const kd_tensor* proj, int q_col, int k_col, int v_col,
                  state->shape[2] == p.dk_pad && state->shape[3] == p.dv_pad, "state must be fp32 [B,heads,%d,%d]", p.dk_pad, p.dv_pad);
   KD_REQUIRE(out->dtype == KD_F32 && is_contiguous(out) && numel(out) == T * heads * vdim, "out must be fp32 [T, heads*vdim]");
   if (T == 0) return KD_OK;
+  KD_REQUIRE((int64_t)p.S * p.ld < (1ll << 31), "delta rule: %d tokens of %lld columns in one call", p.S, (long long)p.ld);
   p.q_scale = (float)(1.0 / sqrt((double)dim));
   void *pp, *pa, *ph, *ps, *po;
   KD_TRY(tensor_ptr(proj, &pp));
@@ -453,6 +724,12 @@ KD_API int kd_delta_rule(const kd_tensor* proj, int q_col, int k_col, int v_col,
   KD_TRY(tensor_ptr(out, &po));
   KD_REQUIRE((reinterpret_cast<uintptr_t>(ps) & 15) == 0, "state must be 16-byte aligned");
   p.a = static_cast<const float*>(pa);
+  const int vb = 4 * dtype_size(proj->dtype);
+  const bool rows_ok = p.ld % 4 == 0 && history->strides[0] % 4 == 0 && history->strides[1] % 4 == 0 &&
+                       reinterpret_cast<uintptr_t>(pp) % vb == 0 && reinterpret_cast<uintptr_t>(ph) % vb == 0;
+  p.vec_q = rows_ok && p.taps <= 4 && dim % 4 == 0 && q_col % 4 == 0 && k_col % 4 == 0;
+  p.vec_v = rows_ok && p.taps <= 4 && vdim % 4 == 0 && v_col % 4 == 0 && kv_heads * dim % 2 == 0;
+  p.vec_a = dim % 4 == 0 && p.ld_a % 4 == 0 && reinterpret_cast<uintptr_t>(pa) % 16 == 0;
   p.state = static_cast<float*>(ps);
   p.o = static_cast<float*>(po);
   if (proj->dtype == KD_BF16) return launch_delta_lpc<__nv_bfloat16>(pp, ph, history->strides[0], history->strides[1], p);
