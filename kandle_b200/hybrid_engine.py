@@ -87,6 +87,8 @@ class _Weights:
 
     def _get(self, name: str, shape) -> np.ndarray:
         a = np.asarray(self.src[name], np.float32)
+        if shape == () and a.size == 1:      # a scalar may be stored as a vector of one
+            a = a.reshape(())
         if tuple(a.shape) != tuple(shape):
             raise ValueError(f"{name} has shape {tuple(a.shape)}, the configuration says {tuple(shape)}")
         return a
