@@ -578,16 +578,19 @@ int kd_moe_linear(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* 
 int kd_latent_prep(const kd_tensor* proj, int q_col, int heads, int dim, int rot_dim, int kv_col, int kv_rank,
                    const kd_tensor* norm_weight, float eps, const kd_tensor* cos, const kd_tensor* sin, const kd_tensor* cache,
                    const kd_tensor* pos_dev, int pos_host, const kd_tensor* dense);
-/* q_abs [B,S,H,width] = (wuk[h]^T q_unrotated, q_rotated, zeros); wuk [H,dim,kv_rank]. */
-int kd_latent_absorb(const kd_tensor* proj, int q_col, int rot_dim, const kd_tensor* wuk, const kd_tensor* q_abs);
+/* q_abs [B,S,H,width] = (wuk[h]^T q_unrotated, q_rotated, zeros); wuk [H,dim,kv_rank].  wuk_t [H,kv_rank,dim], the same
+ * weights the other way round, may be given for the tensor-core form (bf16, dim a multiple of 32). */
+int kd_latent_absorb(const kd_tensor* proj, int q_col, int rot_dim, const kd_tensor* wuk, const kd_tensor* wuk_t, const kd_tensor* q_abs);
 /* Causal attention of the S queries at position pos on over the cache rows; per row and split the unnormalised sum of
  * latents, part_o fp32 [B*S*H, splits, kv_rank], and (running maximum in the log2 domain, sum), part_ml [B*S*H, splits, 2]. */
 int kd_latent_attention(const kd_tensor* q_abs, const kd_tensor* cache, int kv_rank, float scale, const kd_tensor* pos_dev,
                         int pos_host, const kd_tensor* part_o, const kd_tensor* part_ml);
 int kd_latent_attention_splits(int batch, int queries, int heads, int max_seq_len, int* splits_out);
-/* out [T,H*vdim] = wuv_t[h]^T (combined latent sums), wuv_t [H,kv_rank,vdim]; exp(sink[h]) joins the denominator. */
+/* out [T,H*vdim] = wuv_t[h]^T (combined latent sums), wuv_t [H,kv_rank,vdim]; exp(sink[h]) joins the denominator.
+ * wuv [H,vdim,kv_rank] and latents (scratch [T*H, kv_rank]) may be given for the tensor-core form (bf16, kv_rank a
+ * multiple of 32). */
 int kd_latent_values(const kd_tensor* part_o, const kd_tensor* part_ml, const kd_tensor* sink, const kd_tensor* wuv_t,
-                     const kd_tensor* out);
+                     const kd_tensor* wuv, const kd_tensor* latents, const kd_tensor* out);
 /* Prompts and portions with keys and values expanded: kv bf16 [B, pos+S, heads*dim | heads*vdim] = latents x [W_uk; W_uv]^T,
  * the shared rotated key part read from the cache rows; causal from position pos on; sink may be NULL.  tcgen05. */
 int kd_latent_prefill(const kd_tensor* proj, int q_col, int heads, int dim, int rot_dim, const kd_tensor* kv, int vdim,

@@ -8,12 +8,14 @@
 //   kd_latent_attention  split-KV attention over the cache with rows (query, head): partial sums
 //                        sum_j p_j c_j, running maxima and sums per split.
 //   kd_latent_values     combines the splits (the sink enters the denominator here: exp(sink) with no
-//                        key and no value) and applies W_uv per head.
+//                        key and no value) and applies W_uv per head.  In bf16 both per-head products run
+//                        through head_linear_kernel: mma.sync on fragments loaded straight from global
+//                        memory, one latency for a decode step's few rows.
 // This is the decode path, the path of short portions, and the fp32 path.  Long bf16 prompts expand
 // keys and values once and use the tcgen05 prefill kernel (attention_prefill2.cu).
 //
 // bf16 kernel: a CTA owns 16 (or 32) query-head rows and a range of key tiles.  A key tile (64 cache
-// rows) arrives once through a two-stage cp.async ring and serves both products: S = Q K^T reads it
+// rows) arrives once, one bulk copy a row into a two-stage mbarrier ring, and serves both products: S = Q K^T reads it
 // K-major, O += P V reads its first kv_rank columns transposed (ldmatrix.trans).  Warps split S by
 // 4 key groups x 2 halves of the depth, and O by columns.  mma.sync is used on purpose: a decode step
 // has as many query rows as heads, the tcgen05 tile would be 7/8 padding and its 512-column fp32
@@ -139,6 +141,98 @@ latent_absorb_kernel(const T* __restrict__ q, int64_t ld, int q_col, const T* __
   }
 }
 
+// ----------------------------------------------------------------------------- per-head linear (bf16)
+__device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+// out[t, h, n] = sum_k x[t, h, k] W[h, n, k] for 32 tokens a CTA, 8 columns a warp group.  The order of k inside
+// a product is free as long as both operands agree, so a lane loads eight consecutive k of its row (16 bytes)
+// and uses them as the fragments of two k-steps: no shared memory, every load independent of the others.
+// KW warps share a column tile and split K.  Columns from N on (q_abs): the rotated part of x, then zeros.
+struct HeadLinearParams {
+  int T, H, N, K, n_out;
+  int64_t x_t, x_h;           // strides of x
+  int64_t o_t, o_h;           // strides of out
+  int tail_col, tail_len;     // column n >= N of out = x[tail_col + n - N] for n - N < tail_len, else 0
+};
+
+constexpr int HL_WARPS = 4;
+
+template <int KW>
+__global__ void __launch_bounds__(HL_WARPS * 32)
+head_linear_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out, HeadLinearParams p) {
+  constexpr int NT = HL_WARPS / KW;            // column tiles per CTA
+  __shared__ float red[KW > 1 ? HL_WARPS : 1][32][9];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y, t0 = blockIdx.z * 32;
+  const int tile = blockIdx.x * NT + warp / KW, kw = warp % KW;
+  const int n0 = tile * 8, g = lane >> 2, q = lane & 3;
+  const bool product = n0 < p.N;
+  const int per = (p.K / 32 + KW - 1) / KW, k0 = kw * per, k1 = min(p.K / 32, k0 + per);
+  pdl_wait();
+  pdl_trigger();
+  float acc[2][4] = {};
+  if (product) {
+    const __nv_bfloat16* wr = w + ((int64_t)h * p.N + n0 + g) * p.K + q * 8;
+    const __nv_bfloat16* xr[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) xr[i] = x + (int64_t)min(t0 + g + 8 * i, p.T - 1) * p.x_t + (int64_t)h * p.x_h + q * 8;
+#pragma unroll 4
+    for (int k = k0; k < k1; ++k) {
+      const uint4 b = *reinterpret_cast<const uint4*>(wr + k * 32);
+      uint4 a[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const uint4*>(xr[i] + k * 32);
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        mma16816(acc[m], a[2 * m].x, a[2 * m + 1].x, a[2 * m].y, a[2 * m + 1].y, b.x, b.y);
+        mma16816(acc[m], a[2 * m].z, a[2 * m + 1].z, a[2 * m].w, a[2 * m + 1].w, b.z, b.w);
+      }
+    }
+  }
+  if (KW > 1) {
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) red[warp][m * 16 + g + (e >> 1) * 8][q * 2 + (e & 1)] = acc[m][e];
+    __syncthreads();
+    if (kw != 0) return;
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int o = 1; o < KW; ++o) acc[m][e] += red[warp + o][m * 16 + g + (e >> 1) * 8][q * 2 + (e & 1)];
+  }
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = t0 + m * 16 + g + e * 8, n = n0 + q * 2;
+      if (t >= p.T || n >= p.n_out) continue;
+      __nv_bfloat162 v = __floats2bfloat162_rn(acc[m][2 * e], acc[m][2 * e + 1]);
+      if (!product) {
+        const __nv_bfloat16* tail = x + (int64_t)t * p.x_t + (int64_t)h * p.x_h + p.tail_col + (n - p.N);
+        v.x = n - p.N < p.tail_len ? tail[0] : __float2bfloat16_rn(0.f);
+        v.y = n + 1 - p.N < p.tail_len ? tail[1] : __float2bfloat16_rn(0.f);
+      }
+      *reinterpret_cast<__nv_bfloat162*>(out + (int64_t)t * p.o_t + (int64_t)h * p.o_h + n) = v;
+    }
+}
+
+template <int KW>
+static int launch_head_linear(const void* x, const void* w, void* out, const HeadLinearParams& p) {
+  constexpr int NT = HL_WARPS / KW;
+  const int64_t z = (p.T + 31) / 32;
+  KD_REQUIRE(z <= 65535 && p.H <= 65535, "per-head linear: %d tokens in one call", p.T);
+  dim3 grid(((p.n_out + 7) / 8 + NT - 1) / NT, p.H, (unsigned)z);
+  KD_CUDA_CHECK(launch_ex(head_linear_kernel<KW>, grid, dim3(HL_WARPS * 32), 0, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, p));
+  return after_launch("head_linear_kernel");
+}
+
 // ----------------------------------------------------------------------------- attention over cache rows
 struct LatAttnParams {
   int B, S, H, rank, width, max_s, splits;
@@ -152,29 +246,21 @@ struct LatAttnParams {
   int* err;
 };
 
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
 }
 __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
 }
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
 // row stride of the shared-memory tiles: 16 bytes more than a multiple of 128, so that the eight rows
 // of an ldmatrix fall into different banks
 __host__ __device__ constexpr int lat_stride(int width) { return (width + 63) / 64 * 64 + 8; }
 
 constexpr int LAT_THREADS = 256;
 
-// MT: 16-row query tiles per CTA; KT: keys per tile; NT: 8-column output tiles per warp (even).
-template <int MT, int KT, int NT>
+// MT: 16-row query tiles per CTA; KT: keys per tile; NT: 8-column output tiles per warp (even); QR: k-steps of the
+// query tile that a warp keeps in registers (0: it re-reads them from shared memory).
+template <int MT, int KT, int NT, int QR>
 __global__ void __launch_bounds__(LAT_THREADS)
 latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv_bfloat16* __restrict__ cache, LatAttnParams p) {
   constexpr int ROWS = MT * 16;
@@ -189,6 +275,8 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
   float* ss = reinterpret_cast<float*>(ks + 2 * KT * st);                   // [2][ROWS][KT]
   __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(ss + 2 * ROWS * KT); // [ROWS][PST]
   float* al = reinterpret_cast<float*>(ps + ROWS * PST);                    // [ROWS] rescale factors
+  uint64_t* full = reinterpret_cast<uint64_t*>(al + ROWS);                  // [2]
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(full + 2);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int b = blockIdx.z, split = blockIdx.x, row0 = blockIdx.y * ROWS;
@@ -206,22 +294,33 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
 
   const int wc = p.width / 8;                // 16-byte chunks per row
   const __nv_bfloat16* kbase = cache + (int64_t)b * p.cache_b;
+  // one bulk copy per cache row, issued by the lanes of warp 0
   auto load_tile = [&](int t, int buf) {
-    const int k0 = t * KT;
-    for (int i = tid; i < KT * wc; i += LAT_THREADS) {
-      const int r = i / wc, c = i - r * wc;
-      const int key = min(k0 + r, ctx - 1);   // rows past the context repeat the last one and are masked
-      cp_async16(ks + (buf * KT + r) * st + c * 8, kbase + (int64_t)key * p.cache_s + c * 8);
+    if (lane == 0) sm100::mbar_arrive_expect_tx(&full[buf], (uint32_t)(KT * p.width * 2));
+    __syncwarp();
+    for (int r = lane; r < KT; r += 32) {
+      const int key = min(t * KT + r, ctx - 1);   // rows past the context repeat the last one and are masked
+      sm100::bulk_load(ks + (buf * KT + r) * st, kbase + (int64_t)key * p.cache_s, (uint32_t)(p.width * 2), &full[buf]);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (n_t > 0) load_tile(t_begin, 0);
+  if (tid == 0) {
+    sm100::mbar_init(&full[0], 1);
+    sm100::mbar_init(&full[1], 1);
+    *abort_flag = 0;
+    sm100::fence_mbar_init();
+  }
+  __syncthreads();
+  if (warp == 0 && n_t > 0) {
+    load_tile(t_begin, 0);
+    if (n_t > 1) load_tile(t_begin + 1, 1);
+  }
   for (int i = tid; i < ROWS * wc; i += LAT_THREADS) {
     const int r = i / wc, c = i - r * wc;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (row0 + r < p.rows) v = *reinterpret_cast<const uint4*>(q_abs + ((int64_t)b * p.rows + row0 + r) * p.width + c * 8);
     *reinterpret_cast<uint4*>(qs + r * st + c * 8) = v;
   }
+  __syncthreads();
 
   float o[MT][NT][4];
 #pragma unroll
@@ -237,15 +336,20 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
   const int ksteps = p.width / 16;
   const int ks0 = kh * ((ksteps + 1) / 2), ks1 = kh ? ksteps : (ksteps + 1) / 2;
 
+  uint32_t qr[QR > 0 ? QR : 1][MT][4];
+  if (QR > 0) {
+#pragma unroll
+    for (int k = 0; k < QR; ++k)
+      if (k < ks1 - ks0)
+#pragma unroll
+        for (int m = 0; m < MT; ++m) ldsm4(qr[k][m], qs + (m * 16 + (lane & 15)) * st + (ks0 + k) * 16 + (lane >> 4) * 8);
+  }
+
   for (int it = 0; it < n_t; ++it) {
     const int buf = it & 1;
-    if (it + 1 < n_t) {
-      load_tile(t_begin + it + 1, buf ^ 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();
+    // (every warp must come to the same answer before it leaves the loop: a wait that ran out ends all of them)
+    const bool arrived = sm100::mbar_wait(&full[buf], (uint32_t)((it >> 1) & 1), abort_flag, p.err, 701);
+    if (!__syncthreads_and(arrived)) break;
     const __nv_bfloat16* kt = ks + buf * KT * st;
     // S: this warp's keys kg*KG.., depth steps ks0..ks1
     float sacc[MT][KG / 8][4];
@@ -255,17 +359,28 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
       for (int n = 0; n < KG / 8; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) sacc[m][n][e] = 0.f;
-    for (int k = ks0; k < ks1; ++k) {
-      uint32_t a[MT][4], bb[4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) ldsm4(a[m], qs + (m * 16 + (lane & 15)) * st + k * 16 + (lane >> 4) * 8);
+    auto score_step = [&](const uint32_t (&a)[MT][4], int k) {
+      uint32_t bb[4];
       // lanes 0-7 / 8-15: keys 0-7, depth 0-7 / 8-15; lanes 16-31: keys 8-15 (or, with 8 keys, a repeat)
       const int krow = kg * KG + (lane & 7) + (KG == 16 ? (lane >> 4) * 8 : 0);
       ldsm4(bb, kt + krow * st + k * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
-        mma16816(sacc[m][0], a[m], bb[0], bb[1]);
-        if (KG == 16) mma16816(sacc[m][KG / 8 - 1], a[m], bb[2], bb[3]);
+        mma16816(sacc[m][0], a[m][0], a[m][1], a[m][2], a[m][3], bb[0], bb[1]);
+        if (KG == 16) mma16816(sacc[m][KG / 8 - 1], a[m][0], a[m][1], a[m][2], a[m][3], bb[2], bb[3]);
+      }
+    };
+    if (QR > 0) {
+#pragma unroll
+      for (int k = 0; k < QR; ++k)
+        if (k < ks1 - ks0) score_step(qr[k], ks0 + k);
+    } else {
+#pragma unroll 4
+      for (int k = ks0; k < ks1; ++k) {
+        uint32_t a[MT][4];
+#pragma unroll
+        for (int m = 0; m < MT; ++m) ldsm4(a[m], qs + (m * 16 + (lane & 15)) * st + k * 16 + (lane >> 4) * 8);
+        score_step(a, k);
       }
     }
 #pragma unroll
@@ -324,12 +439,13 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
         ldsm4t(bb, kt + (k * 16 + (lane & 15)) * st + col + (lane >> 4) * 8);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          mma16816(o[m][n], a[m], bb[0], bb[1]);
-          mma16816(o[m][n + 1], a[m], bb[2], bb[3]);
+          mma16816(o[m][n], a[m][0], a[m][1], a[m][2], a[m][3], bb[0], bb[1]);
+          mma16816(o[m][n + 1], a[m][0], a[m][1], a[m][2], a[m][3], bb[2], bb[3]);
         }
       }
     }
-    __syncthreads();       // the tile's buffer is refilled by the next iteration's load
+    __syncthreads();       // every warp is done with the tile: its buffer may be refilled
+    if (warp == 0 && it + 2 < n_t) load_tile(t_begin + it + 2, buf);
   }
 
   if (tid % TPR == 0 && row0 + sr < p.rows) {
@@ -490,6 +606,43 @@ latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__
   }
 }
 
+// Combined latents alone, [T*H, rank] bf16: one CTA per (token, head).
+__global__ void __launch_bounds__(128)
+latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ sink, int H, int rank,
+                      int splits, __nv_bfloat16* __restrict__ out) {
+  extern __shared__ float wt[];       // [splits]
+  pdl_wait();
+  pdl_trigger();
+  const int64_t row = blockIdx.x;
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    const float* ml = part_ml + row * splits * 2;
+    const float sk = sink[row % H] * LOG2E;
+    float m = sk, l = 0.f;
+    for (int s = lane; s < splits; s += 32) if (ml[2 * s + 1] > 0.f) m = fmaxf(m, ml[2 * s]);
+    m = warp_max(m);
+    for (int s = lane; s < splits; s += 32) if (ml[2 * s + 1] > 0.f) l += ml[2 * s + 1] * exp2f(ml[2 * s] - m);
+    l = warp_sum(l) + exp2f(sk - m);
+    for (int s = lane; s < splits; s += 32) wt[s] = ml[2 * s + 1] > 0.f ? exp2f(ml[2 * s] - m) / l : 0.f;
+  }
+  __syncthreads();
+  for (int r = threadIdx.x * 4; r < rank; r += blockDim.x * 4) {      // rank is a multiple of 32
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < splits; ++s) {
+      const float w = wt[s];
+      if (w == 0.f) continue;                                          // (an empty split's rows are not initialised)
+      const float4 v = *reinterpret_cast<const float4*>(part_o + (row * splits + s) * rank + r);
+      acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
+    }
+    __nv_bfloat162 a = __floats2bfloat162_rn(acc.x, acc.y), c = __floats2bfloat162_rn(acc.z, acc.w);
+    uint2 u;
+    u.x = *reinterpret_cast<uint32_t*>(&a);
+    u.y = *reinterpret_cast<uint32_t*>(&c);
+    *reinterpret_cast<uint2*>(out + row * rank + r) = u;
+  }
+}
+
 // ----------------------------------------------------------------------------- host side
 static int pos_ptr(const kd_tensor* pos, const int** out) {
   *out = nullptr;
@@ -501,30 +654,33 @@ static int pos_ptr(const kd_tensor* pos, const int** out) {
   return KD_OK;
 }
 
-template <int MT, int KT, int NT>
+template <int MT, int KT, int NT, int QR>
 static int launch_lat(const void* q, const void* cache, const LatAttnParams& p, int smem) {
   static bool configured[64] = {false};
   if (!configured[ctx().device & 63]) {
-    KD_CUDA_CHECK(cudaFuncSetAttribute(latent_attention_bf16_kernel<MT, KT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    KD_CUDA_CHECK(cudaFuncSetAttribute(latent_attention_bf16_kernel<MT, KT, NT, QR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     configured[ctx().device & 63] = true;
   }
   dim3 grid(p.splits, (p.rows + MT * 16 - 1) / (MT * 16), p.B);
-  KD_CUDA_CHECK(launch_ex(latent_attention_bf16_kernel<MT, KT, NT>, grid, dim3(LAT_THREADS), (size_t)smem, (const __nv_bfloat16*)q,
+  KD_CUDA_CHECK(launch_ex(latent_attention_bf16_kernel<MT, KT, NT, QR>, grid, dim3(LAT_THREADS), (size_t)smem, (const __nv_bfloat16*)q,
                           (const __nv_bfloat16*)cache, p));
   return after_launch("latent_attention_bf16_kernel");
 }
 
 static int lat_smem(int width, int mt, int kt) {
   const int st = lat_stride(width), rows = mt * 16;
-  return (rows * st + 2 * kt * st) * 2 + 2 * rows * kt * 4 + rows * (kt + 8) * 2 + rows * 4;
+  return (rows * st + 2 * kt * st) * 2 + 2 * rows * kt * 4 + rows * (kt + 8) * 2 + rows * 4 + 32;
 }
 
 template <int MT, int KT>
 static int launch_lat_nt(const void* q, const void* cache, const LatAttnParams& p, int smem) {
-  if (p.rank <= 128) return launch_lat<MT, KT, 2>(q, cache, p, smem);
-  if (p.rank <= 256) return launch_lat<MT, KT, 4>(q, cache, p, smem);
-  if (p.rank <= 512) return launch_lat<MT, KT, 8>(q, cache, p, smem);
-  return launch_lat<MT, KT, 16>(q, cache, p, smem);
+  // (the depth is split over two warps: 18 k-steps each cover rows of 576 numbers)
+  constexpr int QR = MT == 1 ? 18 : 0;
+  const bool qr = QR > 0 && p.width <= 576;
+  if (p.rank <= 128) return qr ? launch_lat<MT, KT, 2, QR>(q, cache, p, smem) : launch_lat<MT, KT, 2, 0>(q, cache, p, smem);
+  if (p.rank <= 256) return qr ? launch_lat<MT, KT, 4, QR>(q, cache, p, smem) : launch_lat<MT, KT, 4, 0>(q, cache, p, smem);
+  if (p.rank <= 512) return qr ? launch_lat<MT, KT, 8, QR>(q, cache, p, smem) : launch_lat<MT, KT, 8, 0>(q, cache, p, smem);
+  return launch_lat<MT, KT, 16, 0>(q, cache, p, smem);
 }
 
 }  // namespace kd
@@ -577,7 +733,8 @@ KD_API int kd_latent_prep(const kd_tensor* proj, int q_col, int heads, int dim, 
   return after_launch("latent_prep_kernel");
 }
 
-KD_API int kd_latent_absorb(const kd_tensor* proj, int q_col, int rot_dim, const kd_tensor* wuk, const kd_tensor* q_abs) {
+KD_API int kd_latent_absorb(const kd_tensor* proj, int q_col, int rot_dim, const kd_tensor* wuk, const kd_tensor* wuk_t,
+                            const kd_tensor* q_abs) {
   KD_TRY(require_init());
   KD_REQUIRE(proj && wuk && q_abs, "null tensor");
   KD_REQUIRE(proj->ndim == 3 && proj->strides[2] == 1 && proj->strides[0] == proj->strides[1] * proj->shape[1], "proj must be [B,S,N] with evenly spaced rows");
@@ -594,6 +751,17 @@ KD_API int kd_latent_absorb(const kd_tensor* proj, int q_col, int rot_dim, const
   KD_TRY(tensor_ptr(proj, &pp));
   KD_TRY(tensor_ptr(wuk, &pw));
   KD_TRY(tensor_ptr(q_abs, &pq));
+  if (wuk_t) {
+    KD_REQUIRE(wuk_t->ndim == 3 && is_contiguous(wuk_t) && wuk_t->dtype == wuk->dtype && wuk_t->shape[0] == H && wuk_t->shape[1] == rank && wuk_t->shape[2] == dim,
+               "wuk_t must be [H,kv_rank,dim]");
+    void* pt;
+    KD_TRY(tensor_ptr(wuk_t, &pt));
+    if (proj->dtype == KD_BF16 && dim % 32 == 0 && rank % 8 == 0 && (dim + rot_dim) % 8 == 0 && width % 8 == 0 && q_col % 8 == 0 && proj->strides[1] % 8 == 0 &&
+        ((reinterpret_cast<uintptr_t>(pp) | reinterpret_cast<uintptr_t>(pt) | reinterpret_cast<uintptr_t>(pq)) & 15) == 0) {
+      HeadLinearParams hp{(int)T, H, rank, dim, width, proj->strides[1], dim + rot_dim, (int64_t)H * width, width, dim, rot_dim};
+      return launch_head_linear<1>(static_cast<const __nv_bfloat16*>(pp) + q_col, pt, pq, hp);
+    }
+  }
   const int64_t zt = (T + ABS_TOK - 1) / ABS_TOK;
   KD_REQUIRE(zt <= 65535, "kd_latent_absorb: %lld tokens in one call", (long long)T);
   dim3 grid(H, (width + 127) / 128, (unsigned)zt);
@@ -671,7 +839,8 @@ KD_API int kd_latent_attention(const kd_tensor* q_abs, const kd_tensor* cache, i
   return launch_lat_nt<1, 32>(pq, pc, p, lat_smem(p.width, 1, 32));
 }
 
-KD_API int kd_latent_values(const kd_tensor* part_o, const kd_tensor* part_ml, const kd_tensor* sink, const kd_tensor* wuv_t, const kd_tensor* out) {
+KD_API int kd_latent_values(const kd_tensor* part_o, const kd_tensor* part_ml, const kd_tensor* sink, const kd_tensor* wuv_t,
+                            const kd_tensor* wuv, const kd_tensor* latents, const kd_tensor* out) {
   KD_TRY(require_init());
   KD_REQUIRE(part_o && part_ml && sink && wuv_t && out, "null tensor");
   KD_REQUIRE(wuv_t->ndim == 3 && is_contiguous(wuv_t) && is_contiguous(out) && out->dtype == wuv_t->dtype && (out->dtype == KD_BF16 || out->dtype == KD_F32),
@@ -690,6 +859,20 @@ KD_API int kd_latent_values(const kd_tensor* part_o, const kd_tensor* part_ml, c
   KD_TRY(tensor_ptr(sink, &ps));
   KD_TRY(tensor_ptr(wuv_t, &pw));
   KD_TRY(tensor_ptr(out, &pout));
+  if (wuv && latents) {
+    KD_REQUIRE(wuv->ndim == 3 && is_contiguous(wuv) && wuv->dtype == out->dtype && wuv->shape[0] == H && wuv->shape[1] == vdim && wuv->shape[2] == rank, "wuv must be [H,vdim,kv_rank]");
+    KD_REQUIRE(latents->dtype == out->dtype && is_contiguous(latents) && numel(latents) >= T * H * rank, "latents must be [T*H, kv_rank]");
+    void *pl, *pv;
+    KD_TRY(tensor_ptr(latents, &pl));
+    KD_TRY(tensor_ptr(wuv, &pv));
+    if (out->dtype == KD_BF16 && rank % 32 == 0 && vdim % 8 == 0 &&
+        ((reinterpret_cast<uintptr_t>(pl) | reinterpret_cast<uintptr_t>(pv) | reinterpret_cast<uintptr_t>(pout) | reinterpret_cast<uintptr_t>(po)) & 15) == 0) {
+      KD_CUDA_CHECK(launch_ex(latent_combine_kernel, dim3((unsigned)(T * H)), dim3(128), (size_t)splits * 4, (const float*)po, (const float*)pm, (const float*)ps, H, rank, splits, (__nv_bfloat16*)pl));
+      KD_TRY(after_launch("latent_combine_kernel"));
+      HeadLinearParams hp{(int)T, H, vdim, rank, vdim, (int64_t)H * rank, rank, (int64_t)H * vdim, vdim, 0, 0};
+      return launch_head_linear<4>(pl, pv, pout, hp);
+    }
+  }
   const size_t smem = ((size_t)rank * VAL_TOK + VAL_TOK * splits + 8 * VAL_TOK * 32) * 4;
   KD_REQUIRE(smem <= 48 * 1024, "kv_rank=%d with %d splits is too large", rank, splits);
   const int64_t yt = (T + VAL_TOK - 1) / VAL_TOK;

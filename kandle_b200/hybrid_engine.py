@@ -167,14 +167,18 @@ class _LatentAttention:
         self.wukv = None          # [W_uk; W_uv] as stored, for prompts whose keys and values are expanded
         expandable = eng.dtype == "bfloat16" and m.dim in (64, 128) and m.vdim == m.dim and m.rotDim == 64 and m.kvRank % 8 == 0
         if w.random:
-            self.wuk = w.matrix("", (m.heads, m.dim, m.kvRank))
-            self.wuv_t = w.matrix("", (m.heads, m.kvRank, m.vdim))
+            self.wuk, self.wuk_t = w.matrix("", (m.heads, m.dim, m.kvRank)), w.matrix("", (m.heads, m.kvRank, m.dim))
+            self.wuv_t, self.wuv = w.matrix("", (m.heads, m.kvRank, m.vdim)), w.matrix("", (m.heads, m.vdim, m.kvRank))
             if expandable:
                 self.wukv = w.matrix("", (m.heads * (m.dim + m.vdim), m.kvRank))
         else:
             uk, uv = w.host(p + "mix.uk", (m.heads * m.dim, m.kvRank)), w.host(p + "mix.uv", (m.heads * m.vdim, m.kvRank))
             self.wuk = w._put(uk.reshape(m.heads, m.dim, m.kvRank))
             self.wuv_t = w._put(uv.reshape(m.heads, m.vdim, m.kvRank).transpose(0, 2, 1))
+            self.wuk_t = self.wuv = None      # the layouts of the tensor-core forms
+            if eng.dtype == "bfloat16":
+                self.wuk_t = w._put(uk.reshape(m.heads, m.dim, m.kvRank).transpose(0, 2, 1))
+                self.wuv = w._put(uv.reshape(m.heads, m.vdim, m.kvRank))
             if expandable:
                 self.wukv = w._put(np.concatenate([uk, uv], axis=0))
         self.cos, self.sin = eng.rotation(m.rotBase, m.rotDim)
@@ -200,9 +204,10 @@ class _LatentAttention:
         q_abs = ws("q_abs", (B, S, m.heads, width), dt)
         part_o = ws("part_o", (T * m.heads, ns, m.kvRank), "float32")
         part_ml = ws("part_ml", (T * m.heads, ns, 2), "float32")
-        lib.call("kd_latent_absorb", _r(proj3), self.proj.cols["q"], m.rotDim, _r(self.wuk), _r(q_abs))
+        lib.call("kd_latent_absorb", _r(proj3), self.proj.cols["q"], m.rotDim, _r(self.wuk), _r(self.wuk_t), _r(q_abs))
         lib.call("kd_latent_attention", _r(q_abs), _r(cache), m.kvRank, ctypes.c_float(m.scale), _r(pos_dev), pos_host, _r(part_o), _r(part_ml))
-        lib.call("kd_latent_values", _r(part_o), _r(part_ml), _r(self.sink), _r(self.wuv_t), _r(out))
+        latents = ws("latents", (T * m.heads, m.kvRank), dt) if self.wuv is not None else None
+        lib.call("kd_latent_values", _r(part_o), _r(part_ml), _r(self.sink), _r(self.wuv_t), _r(self.wuv), _r(latents), _r(out))
         return out
 
 

@@ -185,10 +185,10 @@ _SIGNATURES = {
     "kd_moe_gather": [_T, _T, _T, _T, ctypes.c_int, _T, _T, _T],
     "kd_moe_linear": [_T, _T, _T, ctypes.c_int, ctypes.c_float, _T],
     "kd_latent_prep": [_T] + [ctypes.c_int] * 6 + [_T, ctypes.c_float, _T, _T, _T, _T, ctypes.c_int, _T],
-    "kd_latent_absorb": [_T, ctypes.c_int, ctypes.c_int, _T, _T],
+    "kd_latent_absorb": [_T, ctypes.c_int, ctypes.c_int, _T, _T, _T],
     "kd_latent_attention": [_T, _T, ctypes.c_int, ctypes.c_float, _T, ctypes.c_int, _T, _T],
     "kd_latent_attention_splits": [ctypes.c_int] * 4 + [ctypes.POINTER(ctypes.c_int)],
-    "kd_latent_values": [_T, _T, _T, _T, _T],
+    "kd_latent_values": [_T] * 7,
     "kd_latent_prefill": [_T] + [ctypes.c_int] * 4 + [_T, ctypes.c_int, _T, ctypes.c_int, _T, ctypes.c_float, ctypes.c_int, _T],
     "kd_delta_rule": [_T] + [ctypes.c_int] * 4 + [_T] + [ctypes.c_int] * 4 + [_T] * 8,
     "kd_delta_state_shape": [ctypes.c_int, ctypes.c_int, ctypes.POINTER(ctypes.c_int), ctypes.POINTER(ctypes.c_int)],
