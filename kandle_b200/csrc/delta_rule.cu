@@ -1,5 +1,5 @@
 // Gated delta rule with one decay per key channel (a linear-attention layer with an [dim, vdim] fp32
-// state per head), prefill and decode in one kernel.
+// state per head): one kernel for prompts and portions, one for a single token.
 //
 // Per head and token:  S <- g S (rows);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q,
 // with q, k, v = silu(short causal convolution of the projections), q and k unit vectors (q also
@@ -575,6 +575,106 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
   }
 }
 
+// ----------------------------------------------------------------------------- one token (decode)
+// The state of a head is read and written once: HBM-bound.  256 threads per (head, 128 value columns): warp r
+// holds rows r RPW .. of the state, a lane four columns; all loads are issued before anything is waited for.
+template <typename T, int RPW>
+__global__ void __launch_bounds__(256)
+delta_step_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_t hist_b, int64_t hist_ld, DeltaParams p) {
+  constexpr bool FAST = sizeof(T) == 2;
+  constexpr int DK = 8 * RPW;
+  __shared__ __align__(16) float qs[DK], ksm[DK], gs[DK], vs[128];
+  __shared__ __align__(16) float part[8][128];
+  __shared__ float red[2][8];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int unit = blockIdx.x, b = unit / p.H, h = unit - b * p.H, hk = h / (p.H / p.Hk);
+  const int col0 = blockIdx.y * 128, col = col0 + lane * 4;
+  const bool cols = col < p.dv_pad;
+  float* srow = p.state + ((int64_t)unit * p.dk_pad + warp * RPW) * p.dv_pad + (cols ? col : 0);
+  float4 s[RPW];
+  // (written a whole step ago, before the launch that the grid-dependency wait is for)
+#pragma unroll
+  for (int i = 0; i < RPW; ++i) s[i] = *reinterpret_cast<const float4*>(srow + (int64_t)i * p.dv_pad);
+  pdl_wait();
+  pdl_trigger();
+  const T* row = proj + (int64_t)b * p.ld;
+  const T* hb = hist + (int64_t)b * hist_b;
+  const int kc = p.Hk * p.dim, halo = p.taps - 1;
+  auto conv = [&](int column, int channel, const float* w) {
+    float y = dr_f<T>(row[column]) * w[halo];
+    for (int k = 0; k < halo; ++k) y = fmaf(dr_f<T>(hb[(int64_t)k * hist_ld + channel]), w[k], y);
+    return y * dr_sigmoid<FAST>(y);
+  };
+  float q = 0.f, k = 0.f;
+  if (tid < p.dim) {                          // dim <= 256
+    const int c = hk * p.dim + tid;
+    q = conv(p.q_col + c, c, p.conv_q + (int64_t)c * p.taps);
+    k = conv(p.k_col + c, kc + c, p.conv_k + (int64_t)c * p.taps);
+    const int a = h * p.dim + tid;
+    gs[tid] = dr_decay<FAST>(p.neg_rate[h], p.a[(int64_t)b * p.ld_a + a] + p.dt_bias[a]);
+  } else if (tid < DK) {
+    gs[tid] = 0.f;
+  }
+  const float sq = warp_sum(q * q), sk = warp_sum(k * k);
+  if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  if (tid < 128) {
+    const int c = h * p.vdim + col0 + tid;
+    vs[tid] = col0 + tid < p.vdim ? conv(p.v_col + c, 2 * kc + c, p.conv_v + (int64_t)c * p.taps) : 0.f;
+  }
+  const float beta = dr_sigmoid<FAST>(dr_f<T>(row[p.b_col + h]));
+  __syncthreads();
+  float nq = 0.f, nk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) { nq += red[0][w]; nk += red[1][w]; }
+  if (tid < DK) {
+    qs[tid] = q * (p.q_scale / sqrtf(nq + 1e-6f));
+    ksm[tid] = k * (1.0f / sqrtf(nk + 1e-6f));
+  }
+  __syncthreads();
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < RPW; ++i) {
+    const float g = gs[warp * RPW + i], kk = ksm[warp * RPW + i];
+    s[i].x *= g; s[i].y *= g; s[i].z *= g; s[i].w *= g;
+    acc.x = fmaf(s[i].x, kk, acc.x); acc.y = fmaf(s[i].y, kk, acc.y); acc.z = fmaf(s[i].z, kk, acc.z); acc.w = fmaf(s[i].w, kk, acc.w);
+  }
+  *reinterpret_cast<float4*>(&part[warp][lane * 4]) = acc;
+  __syncthreads();
+  float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int w = 0; w < 8; ++w) {
+    const float4 x = *reinterpret_cast<const float4*>(&part[w][lane * 4]);
+    u.x += x.x; u.y += x.y; u.z += x.z; u.w += x.w;
+  }
+  const float4 v = *reinterpret_cast<const float4*>(&vs[lane * 4]);
+  u.x = beta * (v.x - u.x); u.y = beta * (v.y - u.y); u.z = beta * (v.z - u.z); u.w = beta * (v.w - u.w);
+  __syncthreads();
+  acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < RPW; ++i) {
+    const float kk = ksm[warp * RPW + i], qq = qs[warp * RPW + i];
+    s[i].x = fmaf(kk, u.x, s[i].x); s[i].y = fmaf(kk, u.y, s[i].y); s[i].z = fmaf(kk, u.z, s[i].z); s[i].w = fmaf(kk, u.w, s[i].w);
+    acc.x = fmaf(s[i].x, qq, acc.x); acc.y = fmaf(s[i].y, qq, acc.y); acc.z = fmaf(s[i].z, qq, acc.z); acc.w = fmaf(s[i].w, qq, acc.w);
+    if (cols) *reinterpret_cast<float4*>(srow + (int64_t)i * p.dv_pad) = s[i];
+  }
+  *reinterpret_cast<float4*>(&part[warp][lane * 4]) = acc;
+  __syncthreads();
+  if (tid < 128 && col0 + tid < p.vdim) {
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) o += part[w][tid];
+    p.o[((int64_t)b * p.H + h) * p.vdim + col0 + tid] = o;
+  }
+}
+
+template <typename T>
+static int launch_delta_step(const void* proj, const void* hist, int64_t hist_b, int64_t hist_ld, const DeltaParams& p) {
+  dim3 grid(p.B * p.H, (p.vdim + 127) / 128);
+  auto k = p.dk_pad == 32 ? delta_step_kernel<T, 4> : p.dk_pad == 64 ? delta_step_kernel<T, 8> : p.dk_pad == 128 ? delta_step_kernel<T, 16> : delta_step_kernel<T, 32>;
+  KD_CUDA_CHECK(launch_ex(k, grid, dim3(256), 0, (const T*)proj, (const T*)hist, hist_b, hist_ld, p));
+  return after_launch("delta_step_kernel");
+}
+
 // ----------------------------------------------------------------------------- output gate + convolution history
 // out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate), one warp per (token, head); the blocks
 // behind them move the last taps - 1 convolution inputs of every channel into the history.
@@ -661,6 +761,7 @@ static int launch_delta(const void* proj, const void* hist, int64_t hist_b, int6
 
 template <typename T>
 static int launch_delta_lpc(const void* proj, const void* hist, int64_t hist_b, int64_t hist_ld, const DeltaParams& p) {
+  if (p.S == 1) return launch_delta_step<T>(proj, hist, hist_b, hist_ld, p);
   if (p.dk_pad == 32) return launch_delta<T, 2>(proj, hist, hist_b, hist_ld, p);
   if (p.dk_pad == 64) return launch_delta<T, 4>(proj, hist, hist_b, hist_ld, p);
   if (p.dk_pad == 128) return launch_delta<T, 8>(proj, hist, hist_b, hist_ld, p);

@@ -248,8 +248,9 @@ KD_API int kd_linear_ex(const kd_tensor* x, const kd_tensor* weight, const kd_te
   if (x->dtype == KD_BF16 && (all & 15) == 0 && K % 8 == 0 && N % 8 == 0 && ldx % 8 == 0 && ldo % (out->dtype == KD_F32 ? 4 : 8) == 0 &&
       (!tail || (n_out % 32 == 0 && (N - n_out) % 4 == 0)) && M < (1ll << 30)) {
     const bool f32 = out->dtype == KD_F32;
-    // a handful of rows: stream the weights through the swapped kernel (its outputs are dense)
-    if (M <= 64 && !residual && ldo == n_out && !(tail && f32) && (f32 || alpha == 1.0f))
+    // a handful of rows: stream the weights through the swapped kernel (its outputs are dense), where its 128-row
+    // weight tiles are enough to fill the GPU or only it can scale the output
+    if (M <= 64 && (alpha != 1.0f || N >= 128ll * (ctx().sm_count / 2)) && !residual && ldo == n_out && !(tail && f32) && (f32 || alpha == 1.0f))
       return gemm_bf16_skinny(px, ldx, pw, K, (int)M, (int)N, (int)K, 1, f32 ? (float*)po : nullptr, f32 ? nullptr : po, 0, alpha, (float*)pt,
                               (int)n_out, tail ? (int)tail->shape[1] : 0);
     if (alpha == 1.0f)

@@ -640,11 +640,13 @@ int gemm_bf16_bias_act(const void* A, int64_t lda, const void* W, int64_t ldw, v
   p.err = ctx().error_flag;
   CUtensorMap ta, tb;
   KD_TRY(make_tmap_bf16_2d(&ta, A, (uint64_t)M, (uint64_t)K, (uint64_t)lda, GEMM_BM, GEMM_BK));
-  if (N >= 256 || epi == 2) {
+  // wide tiles, unless they would leave most of the GPU idle (a few rows, or a narrow output)
+  const int64_t wide = (int64_t)((M + GEMM_BM - 1) / GEMM_BM) * ((N + 255) / 256);
+  if (epi == 2 || (N >= 256 && wide * 2 > ctx().sm_count)) {
     KD_TRY(make_tmap_bf16_2d(&tb, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, 256, GEMM_BK));
     return launch_gemm<256, 4>(ta, tb, p);
   }
-  if (N > 64) {
+  if (N > 64 && wide * 4 > ctx().sm_count) {
     KD_TRY(make_tmap_bf16_2d(&tb, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, 128, GEMM_BK));
     return launch_gemm<128, 6>(ta, tb, p);
   }

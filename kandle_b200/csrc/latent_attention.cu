@@ -15,7 +15,7 @@
 // keys and values once and use the tcgen05 prefill kernel (attention_prefill2.cu).
 //
 // bf16 kernel: a CTA owns 16 (or 32) query-head rows and a range of key tiles.  A key tile (64 cache
-// rows) arrives once, one bulk copy a row into a two-stage mbarrier ring, and serves both products: S = Q K^T reads it
+// rows) arrives once by TMA (128-byte swizzled slabs of 64 columns, two-stage mbarrier ring) and serves both products: S = Q K^T reads it
 // K-major, O += P V reads its first kv_rank columns transposed (ldmatrix.trans).  Warps split S by
 // 4 key groups x 2 halves of the depth, and O by columns.  mma.sync is used on purpose: a decode step
 // has as many query rows as heads, the tcgen05 tile would be 7/8 padding and its 512-column fp32
@@ -262,17 +262,19 @@ constexpr int LAT_THREADS = 256;
 // query tile that a warp keeps in registers (0: it re-reads them from shared memory).
 template <int MT, int KT, int NT, int QR>
 __global__ void __launch_bounds__(LAT_THREADS)
-latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv_bfloat16* __restrict__ cache, LatAttnParams p) {
+latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __grid_constant__ CUtensorMap tmap, LatAttnParams p) {
   constexpr int ROWS = MT * 16;
   constexpr int KG = KT / 4;                 // keys per warp in S (two warps share a key group, each half of the depth)
   constexpr int TPR = LAT_THREADS / ROWS;    // softmax threads per row
   constexpr int KPT = KT / TPR;              // keys per softmax thread
   constexpr int PST = KT + 8;                // row stride of P
-  extern __shared__ __align__(128) uint8_t smem_raw[];
-  const int st = lat_stride(p.width);
-  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);          // [ROWS][st]
-  __nv_bfloat16* ks = qs + ROWS * st;                                       // [2][KT][st]
-  float* ss = reinterpret_cast<float*>(ks + 2 * KT * st);                   // [2][ROWS][KT]
+  constexpr int SLAB = KT * 128;             // bytes of a slab: KT rows of 64 columns
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int st = lat_stride(p.width), slabs = (p.width + 63) / 64;
+  uint8_t* ks = smem;                                                       // [2][slabs][SLAB]
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem + 2 * slabs * SLAB);   // [ROWS][st]
+  float* ss = reinterpret_cast<float*>(qs + ROWS * st);                     // [2][ROWS][KT]
   __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(ss + 2 * ROWS * KT); // [ROWS][PST]
   float* al = reinterpret_cast<float*>(ps + ROWS * PST);                    // [ROWS] rescale factors
   uint64_t* full = reinterpret_cast<uint64_t*>(al + ROWS);                  // [2]
@@ -293,16 +295,12 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
   const int n_t = t_end - t_begin;
 
   const int wc = p.width / 8;                // 16-byte chunks per row
-  const __nv_bfloat16* kbase = cache + (int64_t)b * p.cache_b;
-  // one bulk copy per cache row, issued by the lanes of warp 0
-  auto load_tile = [&](int t, int buf) {
-    if (lane == 0) sm100::mbar_arrive_expect_tx(&full[buf], (uint32_t)(KT * p.width * 2));
-    __syncwarp();
-    for (int r = lane; r < KT; r += 32) {
-      const int key = min(t * KT + r, ctx - 1);   // rows past the context repeat the last one and are masked
-      sm100::bulk_load(ks + (buf * KT + r) * st, kbase + (int64_t)key * p.cache_s, (uint32_t)(p.width * 2), &full[buf]);
-    }
+  auto load_tile = [&](int t, int buf) {     // one thread
+    sm100::mbar_arrive_expect_tx(&full[buf], (uint32_t)(slabs * SLAB));
+    for (int i = 0; i < slabs; ++i) sm100::tma_load_3d(ks + (buf * slabs + i) * SLAB, &tmap, &full[buf], i * 64, t * KT, b);
   };
+  // address of 8 columns (16 bytes) of a row: chunks of a 128-byte row are permuted by the row's low bits
+  auto tile_at = [&](const uint8_t* tile, int row, int col) { return tile + (col >> 6) * SLAB + row * 128 + ((((col >> 3) & 7) ^ (row & 7)) << 4); };
   if (tid == 0) {
     sm100::mbar_init(&full[0], 1);
     sm100::mbar_init(&full[1], 1);
@@ -310,7 +308,7 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
     sm100::fence_mbar_init();
   }
   __syncthreads();
-  if (warp == 0 && n_t > 0) {
+  if (tid == 0 && n_t > 0) {
     load_tile(t_begin, 0);
     if (n_t > 1) load_tile(t_begin + 1, 1);
   }
@@ -350,7 +348,13 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
     // (every warp must come to the same answer before it leaves the loop: a wait that ran out ends all of them)
     const bool arrived = sm100::mbar_wait(&full[buf], (uint32_t)((it >> 1) & 1), abort_flag, p.err, 701);
     if (!__syncthreads_and(arrived)) break;
-    const __nv_bfloat16* kt = ks + buf * KT * st;
+    uint8_t* kt = ks + buf * slabs * SLAB;
+    const int valid = ctx - (t_begin + it) * KT;       // rows past the context hold anything: they must not meet P = 0
+    if (valid < KT) {
+      for (int i = tid; i < (KT - valid) * slabs * 8; i += LAT_THREADS)
+        *reinterpret_cast<uint4*>(kt + (i / ((KT - valid) * 8)) * SLAB + valid * 128 + (i % ((KT - valid) * 8)) * 16) = make_uint4(0, 0, 0, 0);
+      __syncthreads();
+    }
     // S: this warp's keys kg*KG.., depth steps ks0..ks1
     float sacc[MT][KG / 8][4];
 #pragma unroll
@@ -363,7 +367,7 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
       uint32_t bb[4];
       // lanes 0-7 / 8-15: keys 0-7, depth 0-7 / 8-15; lanes 16-31: keys 8-15 (or, with 8 keys, a repeat)
       const int krow = kg * KG + (lane & 7) + (KG == 16 ? (lane >> 4) * 8 : 0);
-      ldsm4(bb, kt + krow * st + k * 16 + ((lane >> 3) & 1) * 8);
+      ldsm4(bb, tile_at(kt, krow, k * 16 + ((lane >> 3) & 1) * 8));
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
         mma16816(sacc[m][0], a[m][0], a[m][1], a[m][2], a[m][3], bb[0], bb[1]);
@@ -436,7 +440,7 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
         const int col = (warp * NT + n) * 8;
         if (col >= p.rank) break;
         uint32_t bb[4];        // keys 0-7 / 8-15 of 8 columns, then of the next 8
-        ldsm4t(bb, kt + (k * 16 + (lane & 15)) * st + col + (lane >> 4) * 8);
+        ldsm4t(bb, tile_at(kt, k * 16 + (lane & 15), col + (lane >> 4) * 8));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma16816(o[m][n], a[m][0], a[m][1], a[m][2], a[m][3], bb[0], bb[1]);
@@ -445,7 +449,7 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __nv
       }
     }
     __syncthreads();       // every warp is done with the tile: its buffer may be refilled
-    if (warp == 0 && it + 2 < n_t) load_tile(t_begin + it + 2, buf);
+    if (tid == 0 && it + 2 < n_t) load_tile(t_begin + it + 2, buf);
   }
 
   if (tid % TPR == 0 && row0 + sr < p.rows) {
@@ -655,25 +659,26 @@ static int pos_ptr(const kd_tensor* pos, const int** out) {
 }
 
 template <int MT, int KT, int NT, int QR>
-static int launch_lat(const void* q, const void* cache, const LatAttnParams& p, int smem) {
+static int launch_lat(const void* q, const CUtensorMap& tmap, const LatAttnParams& p, int smem) {
   static bool configured[64] = {false};
   if (!configured[ctx().device & 63]) {
     KD_CUDA_CHECK(cudaFuncSetAttribute(latent_attention_bf16_kernel<MT, KT, NT, QR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     configured[ctx().device & 63] = true;
   }
   dim3 grid(p.splits, (p.rows + MT * 16 - 1) / (MT * 16), p.B);
-  KD_CUDA_CHECK(launch_ex(latent_attention_bf16_kernel<MT, KT, NT, QR>, grid, dim3(LAT_THREADS), (size_t)smem, (const __nv_bfloat16*)q,
-                          (const __nv_bfloat16*)cache, p));
+  KD_CUDA_CHECK(launch_ex(latent_attention_bf16_kernel<MT, KT, NT, QR>, grid, dim3(LAT_THREADS), (size_t)smem, (const __nv_bfloat16*)q, tmap, p));
   return after_launch("latent_attention_bf16_kernel");
 }
 
 static int lat_smem(int width, int mt, int kt) {
   const int st = lat_stride(width), rows = mt * 16;
-  return (rows * st + 2 * kt * st) * 2 + 2 * rows * kt * 4 + rows * (kt + 8) * 2 + rows * 4 + 32;
+  return 1024 + 2 * ((width + 63) / 64) * kt * 128 + rows * st * 2 + 2 * rows * kt * 4 + rows * (kt + 8) * 2 + rows * 4 + 32;
 }
 
 template <int MT, int KT>
-static int launch_lat_nt(const void* q, const void* cache, const LatAttnParams& p, int smem) {
+static int launch_lat_nt(const void* q, const void* cache_rows, const LatAttnParams& p, int smem) {
+  CUtensorMap cache;
+  KD_TRY(make_tmap_bf16_3d(&cache, cache_rows, (uint64_t)p.B, (uint64_t)p.max_s, (uint64_t)p.width, (uint64_t)p.cache_b, (uint64_t)p.cache_s, KT, 64));
   // (the depth is split over two warps: 18 k-steps each cover rows of 576 numbers)
   constexpr int QR = MT == 1 ? 18 : 0;
   const bool qr = QR > 0 && p.width <= 576;
