@@ -825,7 +825,8 @@ def main():
         import kandle_b200
         from kandle_b200 import hybrid_bench
         kandle_b200.init(0)
-        hybrid_bench.main([s for s in a.hybrid_sizes.split(",") if s], a.hybrid_layers, a.hybrid_batch, a.hybrid_prompt, a.hybrid_steps)
+        hybrid_bench.main([s for s in a.hybrid_sizes.split(",") if s], a.hybrid_layers, a.hybrid_batch, a.hybrid_prompt, a.hybrid_steps,
+                          load_peaks()[0][0])
     elif a.impl == "reference":
         run_reference(a)
     else:

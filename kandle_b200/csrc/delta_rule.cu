@@ -576,52 +576,68 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
 }
 
 // ----------------------------------------------------------------------------- one token (decode)
-// The state of a head is read and written once: HBM-bound.  256 threads per (head, 128 value columns): warp r
-// holds rows r RPW .. of the state, a lane four columns; all loads are issued before anything is waited for.
+// The state of a head is read and written once: HBM-bound.  256 threads per (head, 64 value columns): warp r
+// holds rows r RPW .. of the state, a lane four columns of every second one; all loads are issued before anything
+// is waited for, and three blocks share an SM.
 template <typename T, int RPW>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, RPW <= 16 ? 3 : 2)
 delta_step_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_t hist_b, int64_t hist_ld, DeltaParams p) {
   constexpr bool FAST = sizeof(T) == 2;
   constexpr int DK = 8 * RPW;
-  __shared__ __align__(16) float qs[DK], ksm[DK], gs[DK], vs[128];
-  __shared__ __align__(16) float part[8][128];
+  __shared__ __align__(16) float qs[DK], ksm[DK], gs[DK], vs[64];
+  __shared__ __align__(16) float part[16][64];
   __shared__ float red[2][8];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int unit = blockIdx.x, b = unit / p.H, h = unit - b * p.H, hk = h / (p.H / p.Hk);
-  const int col0 = blockIdx.y * 128, col = col0 + lane * 4;
+  constexpr int NR = RPW / 2;                 // rows a lane: half a warp covers 64 columns of a row
+  const int half = lane >> 4, lcol = (lane & 15) * 4;
+  const int col0 = blockIdx.y * 64, col = col0 + lcol;
   const bool cols = col < p.dv_pad;
-  float* srow = p.state + ((int64_t)unit * p.dk_pad + warp * RPW) * p.dv_pad + (cols ? col : 0);
-  float4 s[RPW];
+  float* srow = p.state + ((int64_t)unit * p.dk_pad + warp * RPW + half) * p.dv_pad + (cols ? col : 0);
+  float4 s[NR];
   // (written a whole step ago, before the launch that the grid-dependency wait is for)
 #pragma unroll
-  for (int i = 0; i < RPW; ++i) s[i] = *reinterpret_cast<const float4*>(srow + (int64_t)i * p.dv_pad);
+  for (int i = 0; i < NR; ++i) s[i] = *reinterpret_cast<const float4*>(srow + (int64_t)(2 * i) * p.dv_pad);
   pdl_wait();
   pdl_trigger();
   const T* row = proj + (int64_t)b * p.ld;
   const T* hb = hist + (int64_t)b * hist_b;
   const int kc = p.Hk * p.dim, halo = p.taps - 1;
-  auto conv = [&](int column, int channel, const float* w) {
-    float y = dr_f<T>(row[column]) * w[halo];
-    for (int k = 0; k < halo; ++k) y = fmaf(dr_f<T>(hb[(int64_t)k * hist_ld + channel]), w[k], y);
+  // (up to four taps: every input and weight is requested before the first is used)
+  auto fetch = [&](int column, int channel, const float* w, float (&x)[4], float (&wt)[4]) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {             // k taps back
+      x[k] = k == 0 ? dr_f<T>(row[column]) : k <= halo ? dr_f<T>(hb[(int64_t)(halo - k) * hist_ld + channel]) : 0.f;
+      wt[k] = k <= halo ? w[halo - k] : 0.f;
+    }
+  };
+  auto finish = [&](int channel, const float* w, const float (&x)[4], const float (&wt)[4]) {
+    float y = fmaf(x[3], wt[3], fmaf(x[2], wt[2], fmaf(x[1], wt[1], x[0] * wt[0])));
+    for (int k = 4; k <= halo; ++k) y = fmaf(dr_f<T>(hb[(int64_t)(halo - k) * hist_ld + channel]), w[halo - k], y);
     return y * dr_sigmoid<FAST>(y);
   };
-  float q = 0.f, k = 0.f;
+  float xq[4], wq[4], xk[4], wk[4], xv[4], wv[4], decay = 0.f, bias = 0.f;
+  const int cq = hk * p.dim + tid, cv = h * p.vdim + col0 + tid, ca = h * p.dim + tid;
+  const bool has_v = tid < 64 && col0 + tid < p.vdim;
   if (tid < p.dim) {                          // dim <= 256
-    const int c = hk * p.dim + tid;
-    q = conv(p.q_col + c, c, p.conv_q + (int64_t)c * p.taps);
-    k = conv(p.k_col + c, kc + c, p.conv_k + (int64_t)c * p.taps);
-    const int a = h * p.dim + tid;
-    gs[tid] = dr_decay<FAST>(p.neg_rate[h], p.a[(int64_t)b * p.ld_a + a] + p.dt_bias[a]);
+    fetch(p.q_col + cq, cq, p.conv_q + (int64_t)cq * p.taps, xq, wq);
+    fetch(p.k_col + cq, kc + cq, p.conv_k + (int64_t)cq * p.taps, xk, wk);
+    decay = p.a[(int64_t)b * p.ld_a + ca];
+    bias = p.dt_bias[ca];
+  }
+  if (has_v) fetch(p.v_col + cv, 2 * kc + cv, p.conv_v + (int64_t)cv * p.taps, xv, wv);
+  const float beta = dr_sigmoid<FAST>(dr_f<T>(row[p.b_col + h]));
+  float q = 0.f, k = 0.f;
+  if (tid < p.dim) {
+    q = finish(cq, p.conv_q + (int64_t)cq * p.taps, xq, wq);
+    k = finish(kc + cq, p.conv_k + (int64_t)cq * p.taps, xk, wk);
+    gs[tid] = dr_decay<FAST>(p.neg_rate[h], decay + bias);
   } else if (tid < DK) {
     gs[tid] = 0.f;
   }
+  if (tid < 64) vs[tid] = has_v ? finish(2 * kc + cv, p.conv_v + (int64_t)cv * p.taps, xv, wv) : 0.f;
   const float sq = warp_sum(q * q), sk = warp_sum(k * k);
   if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
-  if (tid < 128) {
-    const int c = h * p.vdim + col0 + tid;
-    vs[tid] = col0 + tid < p.vdim ? conv(p.v_col + c, 2 * kc + c, p.conv_v + (int64_t)c * p.taps) : 0.f;
-  }
-  const float beta = dr_sigmoid<FAST>(dr_f<T>(row[p.b_col + h]));
   __syncthreads();
   float nq = 0.f, nk = 0.f;
 #pragma unroll
@@ -633,43 +649,43 @@ delta_step_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
   __syncthreads();
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-  for (int i = 0; i < RPW; ++i) {
-    const float g = gs[warp * RPW + i], kk = ksm[warp * RPW + i];
+  for (int i = 0; i < NR; ++i) {
+    const float g = gs[warp * RPW + 2 * i + half], kk = ksm[warp * RPW + 2 * i + half];
     s[i].x *= g; s[i].y *= g; s[i].z *= g; s[i].w *= g;
     acc.x = fmaf(s[i].x, kk, acc.x); acc.y = fmaf(s[i].y, kk, acc.y); acc.z = fmaf(s[i].z, kk, acc.z); acc.w = fmaf(s[i].w, kk, acc.w);
   }
-  *reinterpret_cast<float4*>(&part[warp][lane * 4]) = acc;
+  *reinterpret_cast<float4*>(&part[warp * 2 + half][lcol]) = acc;
   __syncthreads();
   float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-  for (int w = 0; w < 8; ++w) {
-    const float4 x = *reinterpret_cast<const float4*>(&part[w][lane * 4]);
+  for (int w = 0; w < 16; ++w) {
+    const float4 x = *reinterpret_cast<const float4*>(&part[w][lcol]);
     u.x += x.x; u.y += x.y; u.z += x.z; u.w += x.w;
   }
-  const float4 v = *reinterpret_cast<const float4*>(&vs[lane * 4]);
+  const float4 v = *reinterpret_cast<const float4*>(&vs[lcol]);
   u.x = beta * (v.x - u.x); u.y = beta * (v.y - u.y); u.z = beta * (v.z - u.z); u.w = beta * (v.w - u.w);
   __syncthreads();
   acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-  for (int i = 0; i < RPW; ++i) {
-    const float kk = ksm[warp * RPW + i], qq = qs[warp * RPW + i];
+  for (int i = 0; i < NR; ++i) {
+    const float kk = ksm[warp * RPW + 2 * i + half], qq = qs[warp * RPW + 2 * i + half];
     s[i].x = fmaf(kk, u.x, s[i].x); s[i].y = fmaf(kk, u.y, s[i].y); s[i].z = fmaf(kk, u.z, s[i].z); s[i].w = fmaf(kk, u.w, s[i].w);
     acc.x = fmaf(s[i].x, qq, acc.x); acc.y = fmaf(s[i].y, qq, acc.y); acc.z = fmaf(s[i].z, qq, acc.z); acc.w = fmaf(s[i].w, qq, acc.w);
-    if (cols) *reinterpret_cast<float4*>(srow + (int64_t)i * p.dv_pad) = s[i];
+    if (cols) *reinterpret_cast<float4*>(srow + (int64_t)(2 * i) * p.dv_pad) = s[i];
   }
-  *reinterpret_cast<float4*>(&part[warp][lane * 4]) = acc;
+  *reinterpret_cast<float4*>(&part[warp * 2 + half][lcol]) = acc;
   __syncthreads();
-  if (tid < 128 && col0 + tid < p.vdim) {
+  if (tid < 64 && col0 + tid < p.vdim) {
     float o = 0.f;
 #pragma unroll
-    for (int w = 0; w < 8; ++w) o += part[w][tid];
+    for (int w = 0; w < 16; ++w) o += part[w][tid];
     p.o[((int64_t)b * p.H + h) * p.vdim + col0 + tid] = o;
   }
 }
 
 template <typename T>
 static int launch_delta_step(const void* proj, const void* hist, int64_t hist_b, int64_t hist_ld, const DeltaParams& p) {
-  dim3 grid(p.B * p.H, (p.vdim + 127) / 128);
+  dim3 grid(p.B * p.H, (p.vdim + 63) / 64);
   auto k = p.dk_pad == 32 ? delta_step_kernel<T, 4> : p.dk_pad == 64 ? delta_step_kernel<T, 8> : p.dk_pad == 128 ? delta_step_kernel<T, 16> : delta_step_kernel<T, 32>;
   KD_CUDA_CHECK(launch_ex(k, grid, dim3(256), 0, (const T*)proj, (const T*)hist, hist_b, hist_ld, p));
   return after_launch("delta_step_kernel");

@@ -261,7 +261,7 @@ constexpr int LAT_THREADS = 256;
 // MT: 16-row query tiles per CTA; KT: keys per tile; NT: 8-column output tiles per warp (even); QR: k-steps of the
 // query tile that a warp keeps in registers (0: it re-reads them from shared memory).
 template <int MT, int KT, int NT, int QR>
-__global__ void __launch_bounds__(LAT_THREADS)
+__global__ void __launch_bounds__(LAT_THREADS, MT == 1 && KT == 32 && NT <= 8 ? 2 : 1)
 latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __grid_constant__ CUtensorMap tmap, LatAttnParams p) {
   constexpr int ROWS = MT * 16;
   constexpr int KG = KT / 4;                 // keys per warp in S (two warps share a key group, each half of the depth)
@@ -378,6 +378,27 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __gr
 #pragma unroll
       for (int k = 0; k < QR; ++k)
         if (k < ks1 - ks0) score_step(qr[k], ks0 + k);
+    } else if (KG == 8) {
+      // two k-steps per key fragment load, a chain of products each
+      float odd[MT][4] = {};
+#pragma unroll 3
+      for (int k = ks0; k < ks1; k += 2) {
+        const bool two = k + 1 < ks1;
+        uint32_t a[MT][4], c[MT][4], bb[4];
+        ldsm4(bb, tile_at(kt, kg * 8 + (lane & 7), (two ? k + (lane >> 4) : k) * 16 + ((lane >> 3) & 1) * 8));
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          const __nv_bfloat16* qrow = qs + (m * 16 + (lane & 15)) * st + k * 16 + (lane >> 4) * 8;
+          ldsm4(a[m], qrow);
+          ldsm4(c[m], two ? qrow + 16 : qrow);
+          mma16816(sacc[m][0], a[m][0], a[m][1], a[m][2], a[m][3], bb[0], bb[1]);
+          if (two) mma16816(odd[m], c[m][0], c[m][1], c[m][2], c[m][3], bb[2], bb[3]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sacc[m][0][e] += odd[m][e];
     } else {
 #pragma unroll 4
       for (int k = ks0; k < ks1; ++k) {
@@ -680,7 +701,7 @@ static int launch_lat_nt(const void* q, const void* cache_rows, const LatAttnPar
   CUtensorMap cache;
   KD_TRY(make_tmap_bf16_3d(&cache, cache_rows, (uint64_t)p.B, (uint64_t)p.max_s, (uint64_t)p.width, (uint64_t)p.cache_b, (uint64_t)p.cache_s, KT, 64));
   // (the depth is split over two warps: 18 k-steps each cover rows of 576 numbers)
-  constexpr int QR = MT == 1 ? 18 : 0;
+  constexpr int QR = MT == 1 && KT == 64 ? 18 : 0;
   const bool qr = QR > 0 && p.width <= 576;
   if (p.rank <= 128) return qr ? launch_lat<MT, KT, 2, QR>(q, cache, p, smem) : launch_lat<MT, KT, 2, 0>(q, cache, p, smem);
   if (p.rank <= 256) return qr ? launch_lat<MT, KT, 4, QR>(q, cache, p, smem) : launch_lat<MT, KT, 4, 0>(q, cache, p, smem);
@@ -782,7 +803,7 @@ KD_API int kd_latent_attention_splits(int batch, int queries, int heads, int max
   KD_TRY(require_init());
   KD_REQUIRE(splits_out && batch >= 1 && queries >= 1 && heads >= 1 && max_seq_len >= 1, "bad argument");
   const int64_t rows = (int64_t)queries * heads, tiles = batch * ((rows + (rows > 16 ? 31 : 15)) / (rows > 16 ? 32 : 16));
-  int64_t s = ctx().sm_count / tiles, cap = (max_seq_len + 63) / 64;
+  int64_t s = (rows > 16 ? 1 : 2) * ctx().sm_count / tiles, cap = (max_seq_len + 63) / 64;
   if (s > cap) s = cap;
   *splits_out = s < 1 ? 1 : (int)s;
   return KD_OK;
@@ -839,6 +860,8 @@ KD_API int kd_latent_attention(const kd_tensor* q_abs, const kd_tensor* cache, i
     if (lat_smem(p.width, 2, 64) <= limit) return launch_lat_nt<2, 64>(pq, pc, p, lat_smem(p.width, 2, 64));
     if (lat_smem(p.width, 2, 32) <= limit) return launch_lat_nt<2, 32>(pq, pc, p, lat_smem(p.width, 2, 32));
   }
+  // 32-key tiles let two CTAs share an SM: one's softmax runs under the other's products
+  if (kv_rank <= 512 && 2 * (lat_smem(p.width, 1, 32) + 1024) <= limit) return launch_lat_nt<1, 32>(pq, pc, p, lat_smem(p.width, 1, 32));
   if (lat_smem(p.width, 1, 64) <= limit) return launch_lat_nt<1, 64>(pq, pc, p, lat_smem(p.width, 1, 64));
   KD_REQUIRE(lat_smem(p.width, 1, 32) <= limit, "latent rows of %d numbers are too wide", p.width);
   return launch_lat_nt<1, 32>(pq, pc, p, lat_smem(p.width, 1, 32));

@@ -14,10 +14,10 @@ from collections import OrderedDict
 
 import numpy as np
 
-from . import hybrid_engine, lib, synth
+from . import core, lib, synth
 from .backend import CudaEvent
 from .core import Tensor
-from .engine import Qwen3Engine, RandomInit
+from .engine import Qwen3Engine, RandomInit, _r
 from .hybrid_engine import HybridEngine
 from .model_utils.pedorax import PedoraxConfig
 from .model_utils.qwen3 import Qwen3Config
@@ -99,7 +99,66 @@ def _timed(fn, reps: int) -> float:
     return float(np.median(best))
 
 
-def run_size(size: str, layers: int, batch: int, prompt: int, steps: int, profile: bool) -> dict:
+def decode_rooflines(size: str, batch: int, ctx: int, hbm_gbs: float) -> dict:
+    """The HBM-bound kernels of a decode step alone, each over enough operand sets that every launch streams from HBM
+    (one captured graph of 8 launches, replayed), and Qwen3's decode attention beside them."""
+    s = SIZES[size]
+    H, rank, W, E, ff = s["heads"], s["rank"], s["width"], s["experts"], s["ff"]
+    width = (rank + 64 + 15) // 16 * 16
+    out = {}
+
+    def rand(shape, dtype="bfloat16"):
+        t = core.empty(shape, dtype)
+        lib.call("kd_randn", _r(t), ctypes.c_uint64(1), ctypes.c_uint32(0), ctypes.c_float(0.0), ctypes.c_float(0.05), 0, 0, 0)
+        return t
+
+    def measure(name, nbytes, launches):
+        for fn in launches:
+            fn()
+        lib.call("kd_graph_begin")
+        for i in range(8):
+            launches[i % len(launches)]()
+        g = ctypes.c_uint64(0)
+        lib.call("kd_graph_end", ctypes.byref(g))
+        ms = _timed(lambda: lib.call("kd_graph_launch", g), 5) / 8
+        lib.call("kd_graph_destroy", g)
+        out[name] = {"us": round(ms * 1e3, 2), "bytes": int(nbytes), "gbs": round(nbytes / ms / 1e6), "of_measured_hbm": round(nbytes / ms / 1e6 / hbm_gbs, 3)}
+
+    sets = 4
+    caches = [rand((batch, ctx + 64, width)) for _ in range(sets)]
+    q = rand((batch, 1, H, width))
+    n = ctypes.c_int(0)
+    lib.call("kd_latent_attention_splits", batch, 1, H, ctx + 64, ctypes.byref(n))
+    po, pm = core.empty((batch * H, n.value, rank)), core.empty((batch * H, n.value, 2))
+    measure("latent_attention", batch * ctx * (rank + 64) * 2, [
+        (lambda c: lambda: lib.call("kd_latent_attention", _r(q), _r(c), rank, ctypes.c_float(0.07), None, ctx - 1, _r(po), _r(pm)))(c) for c in caches])
+    del caches
+    N = 3 * H * 128 + H + 64 - H % 8
+    proj, dec = rand((batch, 1, N)), rand((batch, H * 128), "float32")
+    conv, vec, big = rand((H * 128, 4), "float32"), rand((H,), "float32"), rand((H * 128,), "float32")
+    states = [core.zeros((batch, H, 128, 128), "float32") for _ in range(sets)]
+    hist, o = core.zeros((batch, 3, 3 * H * 128), "bfloat16"), core.empty((batch, H * 128), "float32")
+    measure("delta_step", 2 * batch * H * 128 * 128 * 4, [
+        (lambda st: lambda: lib.call("kd_delta_rule", _r(proj), 0, H * 128, 2 * H * 128, 3 * H * 128, _r(dec), H, H, 128, 128, _r(conv), _r(conv), _r(conv),
+                                     _r(vec), _r(big), _r(hist), _r(st), _r(o)))(st) for st in states])
+    del states
+    R = batch * s["top"]
+    off = Tensor((np.arange(E + 1) * R // E).astype(np.int32))
+    used = len({int(e) for e in np.arange(R) * E // R}) if R < E else E
+    x, act, y = rand((R, W)), core.empty((R, ff), "bfloat16"), core.empty((R, W), "bfloat16")
+    gus, downs = [rand((E, 2 * ff, W)) for _ in range(2)], [rand((E, W, ff)) for _ in range(2)]
+    measure("expert_gate_up", used * 2 * ff * W * 2, [(lambda w: lambda: lib.call("kd_moe_linear", _r(x), _r(w), _r(off), 4, ctypes.c_float(7.0), _r(act)))(w) for w in gus])
+    measure("expert_down", used * ff * W * 2, [(lambda w: lambda: lib.call("kd_moe_linear", _r(act), _r(w), _r(off), 0, ctypes.c_float(0.0), _r(y)))(w) for w in downs])
+    del gus, downs
+    Hq, Hk = s["qheads"], s["kv_heads"]
+    kv = [(rand((batch, Hk, ctx + 64, 128)), rand((batch, Hk, ctx + 64, 128))) for _ in range(sets)]
+    qq, oo = rand((batch, Hq, 1, 128)), core.empty((batch, Hq, 1, 128), "bfloat16")
+    measure("qwen3_decode_attention", 2 * batch * Hk * ctx * 128 * 2, [
+        (lambda k, v: lambda: lib.call("kd_attention_decode", _r(qq), _r(k), _r(v), None, ctx, ctypes.c_float(0.088), 0, _r(oo)))(k, v) for k, v in kv])
+    return out
+
+
+def run_size(size: str, layers: int, batch: int, prompt: int, steps: int, profile: bool, hbm_gbs: float) -> dict:
     rec = {"size": size, "layers": layers, "batch": batch, "prompt": prompt, "decode_steps": steps}
     ids = Tensor(synth.token_ids(f"hybrid.{size}", (batch, prompt), VOCAB))
     for name, make in engines(size, layers, batch, prompt + 5 * steps + 8):
@@ -125,13 +184,15 @@ def run_size(size: str, layers: int, batch: int, prompt: int, steps: int, profil
         import gc
         gc.collect()
         lib.call("kd_empty_cache")
+    if profile:
+        rec["decode_kernels"] = decode_rooflines(size, batch, prompt, hbm_gbs)
     rec["prefill_ratio"] = round(rec["pedorax"]["prefill_tokens_per_s"] / rec["qwen3"]["prefill_tokens_per_s"], 3)
     rec["decode_ratio"] = round(rec["pedorax"]["decode_tokens_per_s"] / rec["qwen3"]["decode_tokens_per_s"], 3)
     return rec
 
 
-def main(sizes, layers: int, batch: int, prompt: int, steps: int, profile: bool = True) -> None:
+def main(sizes, layers: int, batch: int, prompt: int, steps: int, hbm_gbs: float, profile: bool = True) -> None:
     t0 = time.time()
     for size in sizes:
-        print(json.dumps(run_size(size, layers, batch, prompt, steps, profile)), flush=True)
+        print(json.dumps(run_size(size, layers, batch, prompt, steps, profile, hbm_gbs)), flush=True)
     print(json.dumps({"hybrid_bench_seconds": round(time.time() - t0, 1)}), flush=True)
