@@ -343,11 +343,12 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __gr
         for (int m = 0; m < MT; ++m) ldsm4(qr[k][m], qs + (m * 16 + (lane & 15)) * st + (ks0 + k) * 16 + (lane >> 4) * 8);
   }
 
+  int gave_up = -1;
   for (int it = 0; it < n_t; ++it) {
     const int buf = it & 1;
     // (every warp must come to the same answer before it leaves the loop: a wait that ran out ends all of them)
     const bool arrived = sm100::mbar_wait(&full[buf], (uint32_t)((it >> 1) & 1), abort_flag, p.err, 701);
-    if (!__syncthreads_and(arrived)) break;
+    if (!__syncthreads_and(arrived)) { gave_up = it; break; }
     uint8_t* kt = ks + buf * slabs * SLAB;
     const int valid = ctx - (t_begin + it) * KT;       // rows past the context hold anything: they must not meet P = 0
     if (valid < KT) {
@@ -471,6 +472,10 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __gr
     }
     __syncthreads();       // every warp is done with the tile: its buffer may be refilled
     if (tid == 0 && it + 2 < n_t) load_tile(t_begin + it + 2, buf);
+  }
+  if (gave_up >= 0 && tid == 0) {   // let the copies in flight land before the block leaves its shared memory
+    for (int t = gave_up; t < min(gave_up + 2, n_t); ++t)
+      for (int n = 0; n < (1 << 20) && !sm100::mbar_try_wait(&full[t & 1], (uint32_t)((t >> 1) & 1)); ++n) {}
   }
 
   if (tid % TPR == 0 && row0 + sr < p.rows) {
