@@ -190,7 +190,8 @@ class _LatentAttention:
         cache = cache if cache.shape[0] == B else cache.slice([slice(0, B), slice(None), slice(None)])
         expand = self.wukv is not None and pos_dev is None and S >= eng.expand_from
         # (the layers that read another layer's rows expand the same dense copy)
-        dense = ws(f"latent{self.i if self.own else m.kvFrom}", (T, m.kvRank), dt) if expand and B > 1 and pos_host == 0 else None
+        owner = self if self.own else eng.mixers[m.kvFrom]
+        dense = ws(f"latent{owner.i}", (T, m.kvRank), dt) if expand and owner.wukv is not None and B > 1 and pos_host == 0 else None
         lib.call("kd_latent_prep", _r(proj3), self.proj.cols["q"], m.heads, m.dim, m.rotDim, self.proj.cols.get("dkv", -1), m.kvRank,
                  _r(self.norm), ctypes.c_float(eng.cfg.normEps), _r(self.cos), _r(self.sin), _r(cache), _r(pos_dev), pos_host, _r(dense) if self.own else None)
         out = ws("mixed", (T, m.heads * m.vdim), dt)

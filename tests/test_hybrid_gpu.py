@@ -110,7 +110,7 @@ def test_long_decoding(backend, mixed):
     ("six taps", [(hc.delta(heads=6, kv_heads=2, dim=130, vdim=40, conv=6), None)], {}),
     ("all experts", [(hc.latent(), hc.moe(experts=4, groups=2, keep=2, top=4))], {}),
     ("aligned", [(hc.latent(heads=4, dim=64, rot=32, vdim=64, rank=96), hc.moe(experts=16, top=4, groups=4, ff=64)),
-                 (hc.delta(heads=4, kv_heads=4, dim=64, vdim=64), hc.moe(experts=16, top=2, groups=2, keep=1, ff=32))], dict(width=128, vocab=256)),
+                 (hc.delta(heads=6, kv_heads=3, dim=64, vdim=64), hc.moe(experts=16, top=2, groups=2, keep=1, ff=32))], dict(width=128, vocab=256)),
     ("rows of others", [(hc.latent(), None), (hc.latent(), None), (hc.latent(heads=7, kv_from=0), None), (hc.latent(heads=1, kv_from=1), None),
                         (hc.latent(kv_from=0), None)], {}),
 ])
@@ -141,6 +141,19 @@ def test_expanded_prompts_agree_with_absorbed_ones(backend, dim):
         for cuts in ([390], [130, 128, 70, 62], [64, 1, 100, 225]):
             e = hc.row_errors(hc.run_cut(eng, ids, cuts), ref)
             assert e.max() <= 1.5e-2, (expand_from, cuts, e.max())
+    eng.dispose()
+
+
+def test_expanded_reader_of_rows_that_their_owner_does_not_expand(backend):
+    """The owner's head sizes have no prefill kernel, the reader's do: a batch must expand the cache rows themselves."""
+    cfg = hc.config([(hc.latent(heads=2, dim=32, rot=64, vdim=48, rank=96, scale=0.11), None),
+                     (hc.latent(heads=3, dim=64, rot=64, vdim=64, rank=96, scale=0.11, kv_from=0), None)], width=128)
+    w = hc.weights(cfg, seed=6)
+    ids = hc.tokens(cfg, 2, 200)
+    eng = hc.engine(cfg, w, 2, 200, "bfloat16")
+    assert [m.wukv is not None for m in eng.mixers] == [False, True]
+    e = hc.row_errors(hc.run_cut(eng, ids, [200]), hc.reference(cfg, w, ids))
+    assert e.max() <= 1.5e-2, e.max()
     eng.dispose()
 
 

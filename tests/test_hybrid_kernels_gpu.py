@@ -96,7 +96,7 @@ def _route(logits, top, groups, keep, h):
     return ids.dataAsync(), _get(ws), slots.dataAsync(), off.dataAsync(), xs
 
 
-@pytest.mark.parametrize("E, top, groups, keep", [(8, 2, 4, 3), (64, 6, 8, 4), (12, 1, 1, 1), (6, 4, 6, 4), (300, 8, 10, 5), (64, 8, 32, 32), (4, 4, 2, 2)])
+@pytest.mark.parametrize("E, top, groups, keep", [(8, 3, 4, 2), (64, 6, 8, 4), (12, 1, 1, 1), (6, 4, 6, 4), (300, 8, 10, 5), (64, 8, 32, 32), (4, 4, 2, 2)])
 @pytest.mark.parametrize("T", [1, 37, 700])
 def test_routing_and_expert_order(backend, E, top, groups, keep, T):
     rng = _rng(E, T)
@@ -183,7 +183,7 @@ def _latent_case(B, S, H, rank, rot, vdim, pos, max_s, dtype, splits=None, edit=
     return ref
 
 
-SHAPES = [(1, 1, 6, 96, 32, 32), (2, 1, 16, 512, 64, 128), (1, 1, 40, 64, 16, 24), (2, 3, 5, 40, 8, 12), (1, 7, 20, 256, 64, 64), (1, 2, 3, 600, 64, 16), (1, 1, 33, 9, 2, 5)]
+SHAPES = [(1, 1, 7, 160, 16, 40), (2, 1, 16, 512, 64, 128), (1, 1, 40, 64, 16, 24), (2, 3, 5, 40, 8, 12), (1, 7, 20, 256, 64, 64), (1, 2, 3, 600, 64, 16), (1, 1, 33, 9, 2, 5)]
 
 
 @pytest.mark.parametrize("shape", SHAPES, ids=str)
@@ -222,7 +222,7 @@ def test_sink_from_nothing_to_everything(backend, dtype, value):
     _latent_case(2, 1, 4, 48, 16, 48, 130, 256, dtype, 3, edit)
 
 
-@pytest.mark.parametrize("dim, rot, rank, H", [(128, 64, 512, 16), (32, 32, 96, 6), (24, 16, 48, 3), (7, 2, 9, 2), (64, 0, 40, 3), (96, 32, 64, 5)])
+@pytest.mark.parametrize("dim, rot, rank, H", [(128, 64, 512, 16), (32, 16, 160, 7), (24, 16, 48, 3), (7, 2, 9, 2), (64, 0, 40, 3), (96, 32, 64, 5)])
 @pytest.mark.parametrize("T", [1, 5, 40])
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 def test_absorbed_queries(backend, dim, rot, rank, H, T, dtype):
@@ -283,7 +283,7 @@ def _delta_case(B, S, H, Hk, dim, vdim, taps, dtype, cuts, a_mean=-2.0, a_sd=1.0
         assert np.abs(fin[b] - want).max() <= (1e-4 if dtype == "float32" else 1e-2) * np.abs(want).max()
 
 
-SIZES = [(2, 1, 16, 8, 4), (4, 4, 64, 64, 4), (3, 3, 20, 36, 3), (4, 2, 128, 128, 4), (2, 2, 130, 40, 4), (1, 1, 256, 128, 2), (2, 1, 33, 65, 1), (2, 2, 32, 300, 4), (6, 2, 48, 24, 8), (1, 1, 9, 7, 5)]
+SIZES = [(2, 1, 16, 8, 4), (3, 3, 64, 64, 4), (3, 3, 20, 36, 3), (4, 2, 128, 128, 4), (2, 2, 130, 40, 4), (1, 1, 256, 128, 2), (2, 1, 33, 65, 1), (2, 2, 32, 300, 4), (6, 2, 48, 24, 8), (1, 1, 9, 7, 5)]
 
 
 @pytest.mark.parametrize("size", SIZES, ids=str)
