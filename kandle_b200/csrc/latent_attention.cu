@@ -452,6 +452,10 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __gr
 #pragma unroll
       for (int n = 0; n < NT; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
     }
+    // column tile warp NT + n (+ 1 for the upper lanes): for NT <= 8 a warp's tiles lie in one slab and their chunk
+    // bits differ by an XOR with n alone
+    const uint8_t* vrow = kt + ((warp * NT) >> 3) * SLAB + (lane & 15) * 128;
+    const int vx = ((((warp * NT) & 7) | (lane >> 4)) ^ (lane & 7)) << 4;
 #pragma unroll
     for (int k = 0; k < KT / 16; ++k) {
       uint32_t a[MT][4];
@@ -462,7 +466,8 @@ latent_attention_bf16_kernel(const __nv_bfloat16* __restrict__ q_abs, const __gr
         const int col = (warp * NT + n) * 8;
         if (col >= p.rank) break;
         uint32_t bb[4];        // keys 0-7 / 8-15 of 8 columns, then of the next 8
-        ldsm4t(bb, tile_at(kt, k * 16 + (lane & 15), col + (lane >> 4) * 8));
+        if (NT <= 8) ldsm4t(bb, vrow + k * 2048 + (vx ^ (n << 4)));
+        else ldsm4t(bb, tile_at(kt, k * 16 + (lane & 15), col + (lane >> 4) * 8));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma16816(o[m][n], a[m][0], a[m][1], a[m][2], a[m][3], bb[0], bb[1]);
