@@ -262,6 +262,7 @@ typedef enum kd_epilogue {
                           residual has the output's dtype (bf16, or fp32 residual stream) */
   KD_EPI_CLAMPED_GLU = 4, /* kd_moe_linear: g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit);
                              weight rows interleaved like KD_EPI_SWIGLU */
+  KD_EPI_GEGLU = 5,    /* kd_linear_glu, kd_moe_linear: gelu_tanh(gate) * up; rows interleaved like KD_EPI_SWIGLU */
   KD_EPI_SWIGLU = 2    /* out = silu(x Wg^T) * (x Wu^T) : gate/up `linear`, `silu`, `mul`;
                           weight rows interleave 16 gate rows / 16 up rows per 32-row block      */
 } kd_epilogue;
@@ -570,7 +571,8 @@ int kd_moe_route(const kd_tensor* logits, int top, int groups, int keep, const k
 /* Rows of h in expert order: slots[t,k] = offsets[ids[t,k]] + ranks[t,k], x_sorted[slots[t,k]] = h[t]; offsets [E+1]. */
 int kd_moe_gather(const kd_tensor* h, const kd_tensor* ids, const kd_tensor* ranks, const kd_tensor* counts, int experts,
                   const kd_tensor* slots, const kd_tensor* offsets, const kd_tensor* x_sorted);
-/* out rows of expert e = epilogue(x rows of e * weight[e]^T), weight [E,N,K]; KD_EPI_NONE or KD_EPI_CLAMPED_GLU. */
+/* out rows of expert e = epilogue(x rows of e * weight[e]^T), weight [E,N,K]; KD_EPI_NONE, KD_EPI_CLAMPED_GLU or KD_EPI_GEGLU.
+ * offsets NULL: x holds the same number of rows for every e (several matrices over inputs of their own, one launch). */
 int kd_moe_linear(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* offsets, int epilogue, float limit, const kd_tensor* out);
 /* Rotates the queries' last rot_dim dimensions in place (interleaved pairs) and writes the cache row (normed latent,
  * rotated shared key part) of every token; kv_col < 0: queries only.  proj [B,S,N], cache [B,maxS,width],
@@ -595,18 +597,56 @@ int kd_latent_values(const kd_tensor* part_o, const kd_tensor* part_ml, const kd
  * the shared rotated key part read from the cache rows; causal from position pos on; sink may be NULL.  tcgen05. */
 int kd_latent_prefill(const kd_tensor* proj, int q_col, int heads, int dim, int rot_dim, const kd_tensor* kv, int vdim,
                       const kd_tensor* cache, int kv_rank, const kd_tensor* sink, float scale, int pos, const kd_tensor* out);
-/* Gated delta rule with a decay per key channel; the projections of proj [B,S,N] pass a causal convolution and silu first.
- * decay fp32 [T, heads*dim] (before dt_bias), neg_rate = -exp(A_log) [heads], history [B,taps-1,channels] (q, k, v channels
+/* Gated delta rule; the projections of proj [B,S,N] pass a causal convolution and silu first.
+ * decay fp32 (before dt_bias): one per key channel, [T, heads*dim] with dt_bias [heads*dim], or one per head, [T, >= heads]
+ * with dt_bias [heads]; neg_rate = -exp(A_log) [heads], history [B,taps-1,channels] (q, k, v channels
  * side by side, the inputs before this call), state fp32 [B,heads,rows,cols] as kd_delta_state_shape says, updated in
  * place; out fp32 [T, heads*vdim].  The history is moved on by kd_delta_out, which divides every head's output by its root
- * mean square, multiplies by norm_weight [vdim] and sigmoid(gate), and writes proj's type. */
+ * mean square, multiplies by norm_weight [vdim] and the activated gate (kd_gate), and writes proj's type. */
+typedef enum kd_gate { KD_GATE_SIGMOID = 0, KD_GATE_SILU = 1 } kd_gate;
 int kd_delta_rule(const kd_tensor* proj, int q_col, int k_col, int v_col, int b_col, const kd_tensor* decay, int heads, int kv_heads,
                   int dim, int vdim, const kd_tensor* conv_q, const kd_tensor* conv_k, const kd_tensor* conv_v,
                   const kd_tensor* neg_rate, const kd_tensor* dt_bias, const kd_tensor* history, const kd_tensor* state,
                   const kd_tensor* out);
 int kd_delta_state_shape(int dim, int vdim, int* rows_out, int* cols_out);
-int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, float eps, const kd_tensor* proj,
+int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, float eps, int gate_act, const kd_tensor* proj,
                  int conv_col, int taps, const kd_tensor* history, const kd_tensor* out);
+/* The same norm and gate without a convolution: o fp32 [T, heads*vdim], norm_weight [vdim] (shared by the heads) or
+ * [heads*vdim]; gate and out bf16 or fp32. */
+int kd_gated_head_norm(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, int heads, float eps, int gate_act,
+                       const kd_tensor* out);
+/* Token shift: out[n] = h + (h' - h) mu[n], h' the previous token's row of h [B,S,W]; `last` [B,W] is the row before this
+ * call (zeros at the start of a sequence) and receives the call's last one.  mu fp32 [mixes <= 8, W], out [mixes, B*S, W]. */
+int kd_token_shift(const kd_tensor* h, const kd_tensor* mu, const kd_tensor* last, const kd_tensor* out);
+/* WKV recurrence per head: o = (S + diag(u) k v^T)^T r, then S <- diag(exp(-exp(logit + w0))) S + k v^T.  r, k, v
+ * [B,S,heads*dim] of one layout, logits fp32 [T, heads*dim], w0 and u fp32 [heads*dim], state fp32 [B,heads,rows,cols] as
+ * kd_delta_state_shape(dim, dim) says, updated in place; out fp32 [T, heads*dim].  dim up to 256. */
+int kd_wkv(const kd_tensor* r, const kd_tensor* k, const kd_tensor* v, const kd_tensor* logits, const kd_tensor* w0, const kd_tensor* u,
+           const kd_tensor* state, const kd_tensor* out);
+/* out [M,I] = act(x Wg^T) * (x Wu^T), weight [2I,K] with gate and up rows interleaved in blocks of 16; KD_EPI_SWIGLU or
+ * KD_EPI_GEGLU.  out = tanh(x W^T) for kd_linear_tanh.  bf16 or fp32 throughout. */
+int kd_linear_glu(const kd_tensor* x, const kd_tensor* weight, int epilogue, const kd_tensor* out);
+int kd_linear_tanh(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* out);
+/* x_out = table[ids] (fp32) and h_out, the same in h_out's type.
+ * x_out = x + y / sqrt(mean(y^2) + eps) * norm_weight, y = the sum over splits of y [splits,T,W]; h_out = x_out, or with
+ * final_weight x_out / sqrt(mean(x_out^2) + eps) * final_weight.  Norm weights fp32 [W] as they multiply; x_out may be x. */
+int kd_embed_rows(const kd_tensor* table, const kd_tensor* ids, const kd_tensor* x_out, const kd_tensor* h_out);
+int kd_residual_post_norm(const kd_tensor* x, const kd_tensor* y, const kd_tensor* norm_weight, float eps, const kd_tensor* final_weight,
+                          const kd_tensor* x_out, const kd_tensor* h_out);
+/* Sliding-window grouped-query attention.  kd_attention_head_sizes: the head sizes of the cache rows and of the queries
+ * (bf16 heads up to 128 are padded with zeros to 64 or 128 for the tensor-core kernels; the output has v_size columns a head).
+ * kd_qk_norm_rope_cache: proj [B,S,N] -> q_out [B,S,H,q_size] and the rows at the position of k_cache [B,G,maxS,q_size] and
+ *   v_cache [B,G,maxS,v_size]: one RMS norm over the whole query (key) projection with weights [H*dim] ([G*dim]), then the
+ *   rotation of the first rot_dim dimensions of a head, entry i with i + rot_dim/2; k_col < 0: queries only.
+ * kd_window_attention: query i sees the keys j <= i of the newest `window` (0: all); sink fp32 [H] or NULL: exp(sink) joins the
+ *   denominator.  The bf16 kernels multiply whole 64- or 128-row tiles: cache rows that no query sees get probability
+ *   zero but must be finite. */
+int kd_attention_head_sizes(int dtype, int dim, int vdim, int* q_size_out, int* v_size_out);
+int kd_qk_norm_rope_cache(const kd_tensor* proj, int q_col, int k_col, int v_col, int dim, int vdim, int rot_dim, const kd_tensor* q_norm,
+                          const kd_tensor* k_norm, float eps, const kd_tensor* cos, const kd_tensor* sin, const kd_tensor* k_cache,
+                          const kd_tensor* v_cache, const kd_tensor* pos_dev, int pos_host, const kd_tensor* q_out);
+int kd_window_attention(const kd_tensor* q, const kd_tensor* k_cache, const kd_tensor* v_cache, const kd_tensor* sink, float scale, int window,
+                        const kd_tensor* pos_dev, int pos_host, const kd_tensor* out);
 
 #ifdef __cplusplus
 }

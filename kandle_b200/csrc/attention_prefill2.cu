@@ -34,6 +34,10 @@
 // from the cache rows through a tensor map of its own.  With D = 128, DR = 64 both query tiles and two key
 // tiles take 192 KB, so V has one slot instead of two.  Queries may start behind the first key (a portion
 // of a prompt), and a per-head sink may join the softmax denominator.
+//
+// Sliding window (WIN): the tile loop starts at the first key tile that the CTA's first row sees; keys before a
+// row's window are masked.  Rows may meet tiles of which they see nothing before their first visible key: until then
+// their maximum is held at 0 and their probabilities are exact zeros.
 #include "common.cuh"
 #include "kernels.cuh"
 #include "sm100.cuh"
@@ -69,6 +73,7 @@ struct Fa2Params {
   int B, Hq, Hkv, Sq, Skv;
   int causal;
   int q_off;           // position of query 0 (causal: query i sees keys 0 .. q_off + i)
+  int window;          // WIN: ... of these the newest `window`
   const float* sink;   // [Hq] added to the denominator as exp(sink), or null
   int pair_heads;      // 1: sub-tiles are two heads of one KV group; 0: two consecutive query tiles
   int num_q_tiles;     // 128-row tiles in Sq
@@ -83,7 +88,7 @@ constexpr int FA2_BQ = 128, FA2_BKV = 128, FA2_THREADS = 384;
 constexpr int FA2_NK = 2;
 constexpr int fa2_nv(int D, int DR) { return D == 128 && DR > 0 ? 1 : 2; }
 
-template <int D, int DR>
+template <int D, int DR, bool WIN>
 __global__ void __launch_bounds__(FA2_THREADS, 1)
 flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                                 const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_kr, Fa2Params p) {
@@ -136,6 +141,12 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
       nblk[t] = (kv_end[t] + FA2_BKV - 1) / FA2_BKV;
     }
   }
+  // first key tile of the loop (sub-tile A is never behind B); block numbers below count from it
+  const int j0 = WIN ? max(0, p.q_off + q0[0] - p.window + 1) / FA2_BKV : 0;
+  if (WIN) {
+    nblk[0] = max(0, nblk[0] - j0);
+    nblk[1] = max(0, nblk[1] - j0);
+  }
   const int n_blocks = max(nblk[0], nblk[1]);
 
   if (threadIdx.x == 0) {
@@ -175,15 +186,15 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
         mbar_arrive_expect_tx(&t_full[sk], K_BYTES);
 #pragma unroll
         for (int s = 0; s < SLABS; ++s)
-          tma_load_4d(k_ring + sk * K_BYTES + s * SLAB_BYTES, &tmap_k, &t_full[sk], s * 64, j * FA2_BKV, hk, b);
+          tma_load_4d(k_ring + sk * K_BYTES + s * SLAB_BYTES, &tmap_k, &t_full[sk], s * 64, (j0 + j) * FA2_BKV, hk, b);
 #pragma unroll
         for (int s = SLABS; s < QK_SLABS; ++s)
-          tma_load_4d(k_ring + sk * K_BYTES + s * SLAB_BYTES, &tmap_kr, &t_full[sk], (s - SLABS) * 64, j * FA2_BKV, 0, b);
+          tma_load_4d(k_ring + sk * K_BYTES + s * SLAB_BYTES, &tmap_kr, &t_full[sk], (s - SLABS) * 64, (j0 + j) * FA2_BKV, 0, b);
         if (!mbar_wait(&t_empty[NK + sv], (uint32_t)(((j / NV) & 1) ^ 1), abort_flag, p.err, 402)) break;
         mbar_arrive_expect_tx(&t_full[NK + sv], V_BYTES);
 #pragma unroll
         for (int s = 0; s < SLABS; ++s)
-          tma_load_4d(v_ring + sv * V_BYTES + s * SLAB_BYTES, &tmap_v, &t_full[NK + sv], s * 64, j * FA2_BKV, hk, b);
+          tma_load_4d(v_ring + sv * V_BYTES + s * SLAB_BYTES, &tmap_v, &t_full[NK + sv], s * 64, (j0 + j) * FA2_BKV, hk, b);
       }
     }
   } else if (warp == 9) {
@@ -256,14 +267,16 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
     const uint32_t o_addr = lane_addr + (uint32_t)(256 + t * D);
     const int nb = t ? nblk[1] : nblk[0];
     float m_used = -1e30f, l = 0.f;
+    bool started = false;                   // WIN: this row has seen a key
     bool ok = true;
     for (int j = 0; j < nb; ++j) {
       ok = mbar_wait(&s_full[t], (uint32_t)(j & 1), abort_flag, p.err, 407);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const int kv0 = j * FA2_BKV;
-      const bool masked = (kv0 + FA2_BKV > my_kv_end) || (p.causal && kv0 + FA2_BKV - 1 > p.q_off + my_q0);
+      const int kv0 = (j0 + j) * FA2_BKV;
+      const bool masked = (kv0 + FA2_BKV > my_kv_end) || (p.causal && kv0 + FA2_BKV - 1 > p.q_off + my_q0) ||
+                          (WIN && kv0 + p.window <= p.q_off + my_q0 + FA2_BQ - 1);
       // the whole S row of this thread, once
       uint32_t r[128];
 #pragma unroll
@@ -272,9 +285,10 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
       if (masked) {
         // key kv0 + i is visible to this row iff i <= lim
         const int lim = (p.causal ? min(p.Skv - 1, p.q_off + row) : p.Skv - 1) - kv0;
+        const int low = WIN ? p.q_off + row - p.window + 1 - kv0 : 0;
 #pragma unroll
         for (int i = 0; i < 128; ++i)
-          if (i > lim) r[i] = __float_as_uint(-1e30f);
+          if (i > lim || (WIN && i < low)) r[i] = __float_as_uint(-1e30f);
       }
       float mx0 = -1e30f, mx1 = -1e30f, mx2 = -1e30f, mx3 = -1e30f;
 #pragma unroll
@@ -287,7 +301,10 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
       const float m_blk = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * p.scale_log2;
       float alpha = 1.f;
       bool rescale = false;
-      if (j == 0) {
+      if (WIN && !started) {
+        started = m_blk > -1e30f * p.scale_log2 * 0.5f;      // some key of this tile is visible
+        m_used = started ? m_blk : 0.f;                      // (O and l are still zero: nothing to rescale)
+      } else if (!WIN && j == 0) {
         m_used = m_blk;
       } else if (m_blk - m_used > 8.0f) {      // lazy rescale, see attention_tcgen05.cu
         alpha = fa2_exp2(m_used - m_blk);
@@ -375,16 +392,16 @@ flash_attention_prefill2_kernel(const __grid_constant__ CUtensorMap tmap_q, cons
   }
 }
 
-template <int D, int DR>
+template <int D, int DR, bool WIN = false>
 static int launch_fa2(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tkr, const Fa2Params& p, dim3 grid) {
   constexpr int SMEM = 2 * FA2_BQ * (D + DR) * 2 + FA2_NK * FA2_BKV * (D + DR) * 2 + fa2_nv(D, DR) * FA2_BKV * D * 2 + 1024 + 256;
   static_assert(SMEM <= 227 * 1024, "tiles exceed shared memory");
   static bool configured[64] = {false};   // per device: kd_shutdown + kd_init may move the library to another GPU
   if (!configured[ctx().device & 63]) {
-    KD_CUDA_CHECK(cudaFuncSetAttribute(flash_attention_prefill2_kernel<D, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM));
+    KD_CUDA_CHECK(cudaFuncSetAttribute(flash_attention_prefill2_kernel<D, DR, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM));
     configured[ctx().device & 63] = true;
   }
-  flash_attention_prefill2_kernel<D, DR><<<grid, FA2_THREADS, SMEM, ctx().stream>>>(tq, tk, tv, tkr, p);
+  flash_attention_prefill2_kernel<D, DR, WIN><<<grid, FA2_THREADS, SMEM, ctx().stream>>>(tq, tk, tv, tkr, p);
   return after_launch("flash_attention_prefill2_kernel");
 }
 
@@ -404,6 +421,31 @@ int attention_prefill2(const CUtensorMap& tq, const CUtensorMap& tk, const CUten
   else grid = dim3((p.num_q_tiles + 1) / 2, a.Hq, a.B);
   if (a.D == 128) return launch_fa2<128, 0>(tq, tk, tv, tk, p, grid);
   return launch_fa2<64, 0>(tq, tk, tv, tk, p, grid);
+}
+
+int attention_prefill2_window(const void* q, const void* k, const void* v, void* out, const AttnParams& a, int q_off, int window, const float* sink) {
+  KD_REQUIRE((a.D == 64 || a.D == 128) && a.scale > 0.f && a.Hq % a.Hkv == 0, "attention_prefill2_window: unsupported heads");
+  const int64_t eq[4] = {a.B, a.Hq, a.Sq, a.D}, ek[4] = {a.B, a.Hkv, a.Skv, a.D};
+  CUtensorMap tq, tk, tv;
+  KD_TRY(make_tmap_bhsd(&tq, q, eq, a.sq, FA2_BQ));
+  KD_TRY(make_tmap_bhsd(&tk, k, ek, a.sk, FA2_BKV));
+  KD_TRY(make_tmap_bhsd(&tv, v, ek, a.sv, FA2_BKV));
+  Fa2Params p{};
+  p.B = a.B; p.Hq = a.Hq; p.Hkv = a.Hkv; p.Sq = a.Sq; p.Skv = a.Skv;
+  p.causal = 1;
+  p.q_off = q_off;
+  p.window = window;
+  p.sink = sink;
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.o = static_cast<__nv_bfloat16*>(out);
+  p.so_b = a.so[0]; p.so_h = a.so[1]; p.so_s = a.so[2];
+  p.num_q_tiles = (a.Sq + FA2_BQ - 1) / FA2_BQ;
+  p.err = ctx().error_flag;
+  p.pair_heads = (a.Hq / a.Hkv) % 2 == 0;
+  const dim3 grid = p.pair_heads ? dim3(p.num_q_tiles, a.Hq / 2, a.B) : dim3((p.num_q_tiles + 1) / 2, a.Hq, a.B);
+  const bool win = window > 0 && window < q_off + a.Sq;      // (a window as long as the context hides nothing)
+  if (a.D == 128) return win ? launch_fa2<128, 0, true>(tq, tk, tv, tk, p, grid) : launch_fa2<128, 0>(tq, tk, tv, tk, p, grid);
+  return win ? launch_fa2<64, 0, true>(tq, tk, tv, tk, p, grid) : launch_fa2<64, 0>(tq, tk, tv, tk, p, grid);
 }
 
 }  // namespace kd

@@ -95,6 +95,9 @@ struct FaParams {
   int direct;                  // splits == 1: write O/l as bf16 straight to `o` (no combine kernel)
   int colsplit;                // decode, group <= 8: each softmax warp handles a quarter of the key columns (see kernel)
   int early_kv;                // decode: K/V tiles that do not hold the last position may be fetched before the grid-dependency wait
+  int ctx_add;                 // decode: added to *ctx_ptr (1 when that is the token's position)
+  int window;                  // decode: only the newest `window` keys are seen (0: all)
+  const float* sink;           // decode: [Hq], exp(sink) joins the denominator (null: none)
 };
 
 constexpr int FA_BQ = 128;
@@ -154,7 +157,7 @@ flash_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = blockIdx.z;
-  int h, hk, q0, kv_len, j_begin, j_end, kv_end;
+  int h, hk, q0, kv_len, j_begin, j_end, kv_end, kv_lo = 0;
   // (early_kv: the caller guarantees that the context length and all cache rows but the last
   // position's are older than the launch before this one; see kd_set_pdl)
   if (DECODE && !p.early_kv) pdl_wait();
@@ -163,12 +166,13 @@ flash_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const
     hk = blockIdx.y;
     h = hk;                     // Q tensor map is indexed by (row-in-group, kv head, batch)
     q0 = 0;
-    kv_len = p.ctx_ptr ? *p.ctx_ptr : p.Skv;
+    kv_len = p.ctx_ptr ? *p.ctx_ptr + p.ctx_add : p.Skv;
     kv_len = max(0, min(kv_len, p.Skv));
     kv_end = kv_len;
-    const int n_total = (kv_len + BKV - 1) / BKV;
-    const int per_split = (n_total + p.splits - 1) / p.splits;
-    j_begin = (int)blockIdx.x * per_split;
+    kv_lo = p.window > 0 ? max(0, kv_len - p.window) : 0;      // first key that is seen
+    const int n_total = (kv_len + BKV - 1) / BKV, n_first = kv_lo / BKV;
+    const int per_split = (n_total - n_first + p.splits - 1) / p.splits;
+    j_begin = n_first + (int)blockIdx.x * per_split;
     j_end = min(n_total, j_begin + per_split);
     // the ring takes three K/V tile pairs without anybody having to free a slot; the tile that holds
     // position kv_len - 1 is the last one of the last split
@@ -359,10 +363,10 @@ flash_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const
             tmem_ld_32x16(s_addr + q * QC, sr);
             tmem_wait_ld();
             const int kv0 = (j_begin + j) * BKV + q * QC;
-            if (kv0 + QC > kv_end) {
+            if (kv0 + QC > kv_end || kv0 < kv_lo) {
 #pragma unroll
               for (int i = 0; i < QC; ++i)
-                if (kv0 + i >= kv_len) sr[i] = __float_as_uint(-1e30f);
+                if (kv0 + i >= kv_len || kv0 + i < kv_lo) sr[i] = __float_as_uint(-1e30f);
             }
             float mx0 = -1e30f, mx1 = -1e30f;
 #pragma unroll
@@ -456,7 +460,8 @@ flash_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const
           const int t = (warp - 2) * 32 + lane;
           const int r = t >> 4, cw = D / 16, c0 = (t & 15) * cw;
           if (r < p.group) {
-            const float lsum = xl[r] + xl[32 + r] + xl[64 + r] + xl[96 + r];
+            float lsum = xl[r] + xl[32 + r] + xl[64 + r] + xl[96 + r];
+            if (p.direct && p.sink) lsum += fast_exp2(fmaf(p.sink[hk * p.group + r], 1.4426950408889634f, -xmu[r]));
             float acc[D / 16];
 #pragma unroll
             for (int i = 0; i < cw; ++i)
@@ -500,13 +505,13 @@ flash_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const
       const int kv0 = (j_begin + j) * BKV;
       // Only the diagonal block of a causal tile and the last (ragged) key block need masking;
       // the test is hoisted so that the common path carries no per-element predicates.
-      if ((kv0 + BKV > kv_end) || (p.causal && kv0 + BKV - 1 > q0)) {
+      if ((kv0 + BKV > kv_end) || (p.causal && kv0 + BKV - 1 > q0) || (DECODE && kv0 < kv_lo)) {
 #pragma unroll
         for (int c = 0; c < NCH; ++c)
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int col = kv0 + wg * CW + c * 32 + i;
-            if (col >= kv_len || (p.causal && col > row)) sr[c][i] = __float_as_uint(-1e30f);
+            if (col >= kv_len || (p.causal && col > row) || (DECODE && col < kv_lo)) sr[c][i] = __float_as_uint(-1e30f);
           }
       }
       float mx0 = -1e30f, mx1 = -1e30f;
@@ -602,6 +607,7 @@ flash_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const
       if (DECODE && p.direct) {
         // a single split holds the whole key range: normalise and store the real rows directly
         const bool valid = row_in_tile < p.group;
+        if (p.sink && valid) l += fast_exp2(fmaf(p.sink[hk * p.group + row_in_tile], 1.4426950408889634f, -m_used));
         const float inv_l = 1.0f / l;
         __nv_bfloat16* orow = p.o + (int64_t)b * p.so_b + (int64_t)(hk * p.group + row_in_tile) * p.so_h;
 #pragma unroll 1
@@ -750,10 +756,10 @@ int attention_tc_try(const kd_tensor* q, const kd_tensor* k, const kd_tensor* v,
 }
 
 // ----------------------------------------------------------------------------- split-KV combine
-// out[b, h, :] = sum_s 2^(m_s - M) O_s / sum_s 2^(m_s - M) l_s,  M = max_s m_s.
+// out[b, h, :] = sum_s 2^(m_s - M) O_s / (sum_s 2^(m_s - M) l_s + exp(sink_h) 2^-M),  M = max_s m_s.
 // One warp per (batch, query head); lanes stride over the head dimension.
 __global__ void decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                      __nv_bfloat16* __restrict__ out, int64_t so_b, int64_t so_h, int B, int Hkv,
+                                      const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int64_t so_b, int64_t so_h, int B, int Hkv,
                                       int group, int splits, int D) {
   pdl_wait();
   pdl_trigger();
@@ -765,7 +771,8 @@ __global__ void decode_combine_kernel(const float* __restrict__ part_o, const fl
   const int64_t base = ((int64_t)b * Hkv + hk) * splits;
   float M = -1e30f;
   for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[((base + s) * group + r) * 2]);
-  float denom = 0.f;
+  if (sink) M = fmaxf(M, sink[h] * 1.4426950408889634f);
+  float denom = sink ? exp2f(fmaf(sink[h], 1.4426950408889634f, -M)) : 0.f;
   float acc[8];
 #pragma unroll
   for (int i = 0; i < 8; ++i) acc[i] = 0.f;
@@ -871,8 +878,52 @@ int attention_decode(const kd_tensor* q, const kd_tensor* k, const kd_tensor* v,
   if (p.direct) return KD_OK;
   const int warps = B * Hq;
   KD_CUDA_CHECK(launch_ex(decode_combine_kernel, dim3((warps * 32 + 255) / 256), dim3(256), 0, (const float*)p.part_o,
-                          (const float*)p.part_ml, static_cast<__nv_bfloat16*>(po), (int64_t)out->strides[0],
+                          (const float*)p.part_ml, (const float*)nullptr, static_cast<__nv_bfloat16*>(po), (int64_t)out->strides[0],
                           (int64_t)out->strides[1], B, Hkv, group, splits, D));
+  return after_launch("decode_combine_kernel");
+}
+
+// The newest `window` keys up to a position (kernels.cuh).
+int attention_decode_window(const void* q, const void* k, const void* v, void* out, const WindowDecode& d) {
+  const int group = d.H / d.G, pairs = d.B * d.G;
+  KD_REQUIRE(group <= 16 && d.H % d.G == 0 && (d.D == 64 || d.D == 128) && d.scale > 0.f, "attention_decode_window: unsupported heads");
+  // as many splits as fill the GPU, of two tiles at least
+  const int span = d.window > 0 && d.window < d.max_s ? d.window : d.max_s;
+  const int tiles = (span + FA_DEC_BKV - 1) / FA_DEC_BKV + 1;
+  int splits = 2 * ctx().sm_count / (pairs > 0 ? pairs : 1);
+  if (splits > (tiles + 1) / 2) splits = (tiles + 1) / 2;
+  if (splits < 1) splits = 1;
+  if (splits > 1024) splits = 1024;
+  void* scratch = nullptr;
+  KD_TRY(get_workspace(attention_decode_scratch_bytes(d.B, d.G, group, splits, d.D), &scratch));
+  const int64_t eq[4] = {d.B, d.G, group, d.D}, sq[3] = {(int64_t)d.H * d.D, (int64_t)group * d.D, d.D};
+  const int64_t ek[4] = {d.B, d.G, d.max_s, d.D};
+  CUtensorMap tq, tk, tv;
+  KD_TRY(make_tmap_bhsd(&tq, q, eq, sq, 16));
+  KD_TRY(make_tmap_bhsd(&tk, k, ek, d.kc, FA_DEC_BKV));
+  KD_TRY(make_tmap_bhsd(&tv, v, ek, d.vc, FA_DEC_BKV));
+  FaParams p{};
+  p.B = d.B; p.Hq = d.H; p.Hkv = d.G; p.Sq = group; p.Skv = d.pos_dev ? d.max_s : d.pos_host + 1;
+  p.scale_log2 = d.scale * 1.4426950408889634f;
+  p.err = ctx().error_flag;
+  p.ctx_ptr = d.pos_dev;
+  p.ctx_add = 1;
+  p.window = d.window;
+  p.sink = d.sink;
+  p.splits = splits;
+  p.group = group;
+  p.part_o = static_cast<float*>(scratch);
+  p.part_ml = p.part_o + (size_t)pairs * splits * group * d.D;
+  p.colsplit = group <= 8;
+  p.direct = splits == 1;
+  p.o = static_cast<__nv_bfloat16*>(out);
+  p.so_b = (int64_t)d.H * d.D; p.so_h = d.D; p.so_s = d.D;
+  dim3 grid(splits, d.G, d.B);
+  if (d.D == 128) KD_TRY((launch_fa<128, true>(tq, tk, tv, p, grid)));
+  else KD_TRY((launch_fa<64, true>(tq, tk, tv, p, grid)));
+  if (p.direct) return KD_OK;
+  KD_CUDA_CHECK(launch_ex(decode_combine_kernel, dim3((d.B * d.H * 32 + 255) / 256), dim3(256), 0, (const float*)p.part_o, (const float*)p.part_ml, d.sink,
+                          p.o, p.so_b, p.so_h, d.B, d.G, group, splits, d.D));
   return after_launch("decode_combine_kernel");
 }
 

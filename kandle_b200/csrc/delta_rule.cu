@@ -1,5 +1,5 @@
-// Gated delta rule with one decay per key channel (a linear-attention layer with an [dim, vdim] fp32
-// state per head): one kernel for prompts and portions, one for a single token.
+// Gated delta rule with one decay per key channel or per head (a linear-attention layer with an
+// [dim, vdim] fp32 state per head): one kernel for prompts and portions, one for a single token.
 //
 // Per head and token:  S <- g S (rows);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q,
 // with q, k, v = silu(short causal convolution of the projections), q and k unit vectors (q also
@@ -28,11 +28,12 @@
 // (the state is read and written once per token: 8 dim vdim bytes per head and sequence).
 #include "common.cuh"
 #include "kernels.cuh"
+#include "recurrence.cuh"
 
 namespace kd {
 
-constexpr int DR_CONSUMERS = 8, DR_HELPERS = 8;
-constexpr int DR_THREADS = (DR_CONSUMERS + DR_HELPERS) * 32;
+constexpr int DR_CONSUMERS = REC_CONSUMERS, DR_HELPERS = REC_HELPERS;
+constexpr int DR_THREADS = REC_THREADS;
 constexpr int DR_TB = 16;          // tokens per block
 constexpr int DR_MAX_TAPS = 8;
 
@@ -47,12 +48,13 @@ struct DeltaParams {
   int64_t ld_a;                    // row stride of the decay logits
   float q_scale;
   int vec_q, vec_v, vec_a;         // rows allow four-channel vector loads (q and k, v, decay logits)
-  const float* a;                  // [T, H*dim] decay logits (before dt_bias)
+  int head_decay;                  // one decay per head instead of one per key channel
+  const float* a;                  // [T, H*dim] or [T, H] decay logits (before dt_bias)
   const float* conv_q;             // [Hk*dim, taps]
   const float* conv_k;
   const float* conv_v;             // [H*vdim, taps]
   const float* neg_rate;           // [H] -exp(A_log)
-  const float* dt_bias;            // [H*dim]
+  const float* dt_bias;            // [H*dim] or [H]
   float* state;
   float* o;                        // [T, H*vdim]
 };
@@ -61,64 +63,14 @@ struct DeltaParams {
 // the end of every four tokens [TB/4][dk], v [TB][dv], step sizes and flags [TB].
 __host__ __device__ constexpr int delta_unit_floats(int dk, int dv) { return DR_TB * (4 * dk + dv) + (DR_TB / 4) * dk + 2 * DR_TB; }
 
-template <typename T> __device__ __forceinline__ float dr_f(T v);
-template <> __device__ __forceinline__ float dr_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float dr_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  float2 d;
-  asm("{\n\t.reg .b64 a, b, c, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\t"
-      "fma.rn.f32x2 d, a, b, c;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
-  return d;
-}
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
-  float2 d;
-  asm("{\n\t.reg .b64 a, b, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmul.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
-  return d;
-}
-
-// In bf16 mode (FAST) the elementary functions are the special-function unit's, accurate to a few fp32
-// roundings for these arguments; the fp32 mode uses the accurate library functions.
-__device__ __forceinline__ float ex2f(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ float rcpf(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-constexpr float DR_LOG2E = 1.4426950408889634f;
-template <bool FAST> __device__ __forceinline__ float dr_sigmoid(float x) {
-  return FAST ? rcpf(1.0f + ex2f(-DR_LOG2E * x)) : 1.0f / (1.0f + expf(-x));
-}
 // exp(rate softplus(x))
 template <bool FAST> __device__ __forceinline__ float dr_decay(float rate, float x) {
   if (FAST) {
-    const float z = DR_LOG2E * x;
+    const float z = REC_LOG2E * x;
     return ex2f(rate * (fmaxf(z, 0.f) + __log2f(1.0f + ex2f(-fabsf(z)))));
   }
   return expf(rate * (fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)))));
 }
-
-// Four consecutive channels of a row as they lie in memory.
-template <typename T> struct Raw4;
-template <> struct Raw4<__nv_bfloat16> {
-  uint2 u;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { u = *reinterpret_cast<const uint2*>(p); }
-  __device__ __forceinline__ void get(float (&v)[4]) const {
-    v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
-    v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
-  }
-};
-template <> struct Raw4<float> {
-  float4 f;
-  __device__ __forceinline__ void load(const float* p) { f = *reinterpret_cast<const float4*>(p); }
-  __device__ __forceinline__ void get(float (&v)[4]) const { v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
-};
 
 // The inputs of one short convolution at four tokens: where they are and how to read them.
 template <typename T>
@@ -189,7 +141,7 @@ __device__ __forceinline__ void conv_finish(const ConvSource<T>& cs, int c, cons
 #pragma unroll
   for (int q = 0; q < 4; ++q)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) y[q][e] = c < cs.nc && cs.t + q < cs.S ? acc[q][e] * dr_sigmoid<FAST>(acc[q][e]) : 0.f;
+    for (int e = 0; e < 4; ++e) y[q][e] = c < cs.nc && cs.t + q < cs.S ? acc[q][e] * rec_sigmoid<FAST>(acc[q][e]) : 0.f;
 }
 
 // Element by element, for sizes or strides that allow no vector loads and for more taps.
@@ -202,9 +154,9 @@ __device__ __forceinline__ void conv_slow(const ConvSource<T>& cs, int c, float 
       if (c + e < cs.nc && cs.t + q < cs.S)
         for (int k = 0; k < cs.taps; ++k) {
           const int tt = cs.t + q - halo + k;
-          acc = fmaf(dr_f<T>(tt >= 0 ? cs.row0[tt * cs.ld + c + e] : cs.hist[(tt + halo) * cs.hist_ld + c + e]), cs.w[(int64_t)(c + e) * cs.taps + k], acc);
+          acc = fmaf(rec_f<T>(tt >= 0 ? cs.row0[tt * cs.ld + c + e] : cs.hist[(tt + halo) * cs.hist_ld + c + e]), cs.w[(int64_t)(c + e) * cs.taps + k], acc);
         }
-      y[q][e] = acc * dr_sigmoid<FAST>(acc);
+      y[q][e] = acc * rec_sigmoid<FAST>(acc);
     }
 }
 
@@ -225,9 +177,6 @@ __device__ __forceinline__ void unit_scale(const float (&y)[CH][4][4], float sca
 #pragma unroll
   for (int q = 0; q < 4; ++q) inv[q] = FAST ? scale * rsqrtf(ss[q] + 1e-6f) : scale / sqrtf(ss[q] + 1e-6f);
 }
-
-// Decays below this are applied to the state at once; products of four larger ones keep 1 / P in range.
-constexpr float DR_SMALL_DECAY = 1e-6f;
 
 template <typename T, int LPC>
 __global__ void __launch_bounds__(DR_THREADS, 1)
@@ -268,7 +217,12 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
       const int c0 = lane * 4;
       Raw4<T> raw[7];
       float g[CH][4][4];
-      const float* a = p.a + ((int64_t)b * p.S + t) * p.ld_a + h * p.dim;
+      const float* a = p.a + ((int64_t)b * p.S + t) * p.ld_a + (p.head_decay ? h : h * p.dim);
+      float ah[4] = {0.f, 0.f, 0.f, 0.f};
+      if (p.head_decay) {
+#pragma unroll
+        for (int q = 0; q < 4; ++q) ah[q] = a[(t + q < p.S ? q : 0) * p.ld_a];
+      } else
 #pragma unroll
       for (int i = 0; i < CH; ++i) {
         const int c = i * 128 + c0;
@@ -288,6 +242,18 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
       // decays
       const float rate = p.neg_rate[h];
       float least = 1.f;
+      if (p.head_decay) {
+        const float bias = __ldg(p.dt_bias + h);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          ah[q] = t + q < p.S ? dr_decay<FAST>(rate, ah[q] + bias) : 1.f;
+          least = fminf(least, ah[q]);
+#pragma unroll
+          for (int i = 0; i < CH; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) g[i][q][e] = i * 128 + c0 + e < p.dim ? ah[q] : 1.f;
+        }
+      } else
 #pragma unroll
       for (int i = 0; i < CH; ++i) {
         const int c = i * 128 + c0;
@@ -305,14 +271,14 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
       // running products of the decays since the last one that was applied directly (or the group's start);
       // g becomes that product, d holds what to multiply the state with where a token is flagged
       bool flag[4] = {false, false, false, false};
-      if (__any_sync(0xffffffffu, least < DR_SMALL_DECAY)) {
+      if (__any_sync(0xffffffffu, least < REC_SMALL_DECAY)) {
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
           bool small = false;
 #pragma unroll
           for (int i = 0; i < CH; ++i)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) small |= g[i][q][e] < DR_SMALL_DECAY;
+            for (int e = 0; e < 4; ++e) small |= g[i][q][e] < REC_SMALL_DECAY;
           flag[q] = __any_sync(0xffffffffu, small);
         }
       }
@@ -394,7 +360,7 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
       }
       if (lane < 4) {
         float* beta = v + DR_TB * dvc;
-        beta[2 * (grp * 4 + lane)] = t + lane < p.S ? dr_sigmoid<FAST>(dr_f<T>(seq[(int64_t)(t + lane) * p.ld + p.b_col + h])) : 0.f;
+        beta[2 * (grp * 4 + lane)] = t + lane < p.S ? rec_sigmoid<FAST>(rec_f<T>(seq[(int64_t)(t + lane) * p.ld + p.b_col + h])) : 0.f;
         beta[2 * (grp * 4 + lane) + 1] = (lane == 0 ? flag[0] : lane == 1 ? flag[1] : lane == 2 ? flag[2] : flag[3]) ? 1.f : 0.f;
       }
     }
@@ -426,65 +392,13 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
   const bool active = live && col < p.dv_pad;
   float2 s[8][8];                              // [column][row pair]
   float* srow = nullptr;
-#pragma unroll
-  for (int c = 0; c < 8; ++c)
-#pragma unroll
-    for (int r = 0; r < 8; ++r) s[c][r] = make_float2(0.f, 0.f);
   // (the state was last written a whole step ago, before the launch that the grid-dependency wait is for)
-  if (active) {
-    srow = p.state + ((int64_t)unit * p.dk_pad + j * 4) * p.dv_pad + col;
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-#pragma unroll
-        for (int w = 0; w < 2; ++w) {
-          const float4 v = *reinterpret_cast<const float4*>(srow + (int64_t)(i * LPC * 4 + e) * p.dv_pad + w * 4);
-          const float vv[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            if (e & 1) s[w * 4 + c][i * 2 + (e >> 1)].y = vv[c];
-            else s[w * 4 + c][i * 2 + (e >> 1)].x = vv[c];
-          }
-        }
-  }
+  if (active) srow = p.state + ((int64_t)unit * p.dk_pad + j * 4) * p.dv_pad + col;
+  state_load<LPC>(s, srow, p.dv_pad);
   pdl_wait();
   pdl_trigger();
   block_barrier();
 
-  auto scale_state = [&](const float4* d4) {
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float4 d = d4[i * LPC];
-#pragma unroll
-      for (int c = 0; c < 8; ++c) {
-        s[c][2 * i] = mul2(s[c][2 * i], make_float2(d.x, d.y));
-        s[c][2 * i + 1] = mul2(s[c][2 * i + 1], make_float2(d.z, d.w));
-      }
-    }
-  };
-  // Sums x and y over the group's lanes; lane j ends with columns own .. own + OWN - 1 in [0, OWN).
-  auto group_sums = [&](float (&x)[8], float (&y)[8]) {
-    int n = 8;
-#pragma unroll
-    for (int m = LPC / 2; m > 0; m >>= 1) {
-      if (n > 1) {
-        n >>= 1;
-        const bool up = j & m;
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-          if (i < n) {
-            const float sx = up ? x[i] : x[i + n], kx = up ? x[i + n] : x[i];
-            const float sy = up ? y[i] : y[i + n], ky = up ? y[i + n] : y[i];
-            x[i] = kx + __shfl_xor_sync(0xffffffffu, sx, m);
-            y[i] = ky + __shfl_xor_sync(0xffffffffu, sy, m);
-          }
-      } else {
-        x[0] += __shfl_xor_sync(0xffffffffu, x[0], m);
-        y[0] += __shfl_xor_sync(0xffffffffu, y[0], m);
-      }
-    }
-  };
   const int b = live ? unit / p.H : 0, h = live ? unit - b * p.H : 0;
   float po[8];                                 // this lane's share of the previous token's output
 #pragma unroll
@@ -511,7 +425,7 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
         float v[OWN];
 #pragma unroll
         for (int i = 0; i < OWN; ++i) v[i] = vb[t * dvc + lcol + own + i];
-        if (bf.y != 0.f) scale_state(reinterpret_cast<const float4*>(base + (3 * DR_TB + t) * DK) + j);
+        if (bf.y != 0.f) state_scale<LPC>(s, reinterpret_cast<const float4*>(base + (3 * DR_TB + t) * DK) + j);
         float2 acc[8];
 #pragma unroll
         for (int c = 0; c < 8; ++c) acc[c] = make_float2(0.f, 0.f);
@@ -527,7 +441,7 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
 #pragma unroll
         for (int c = 0; c < 8; ++c) pr[c] = acc[c].x + acc[c].y;
         // the previous token's output leaves here: its shuffles fill the wait for this token's
-        group_sums(pr, po);
+        group_sums<LPC>(j, pr, po);
         store_out(orow + (int64_t)(t0 + t - 1) * o_ld, t0 + t > 0);
 #pragma unroll
         for (int i = 0; i < OWN; ++i) pr[i] = bf.x * (v[i] - pr[i]);
@@ -550,29 +464,17 @@ delta_rule_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
         }
 #pragma unroll
         for (int c = 0; c < 8; ++c) po[c] = acc[c].x + acc[c].y;
-        if ((t & 3) == 3 || t + 1 == n) scale_state(reinterpret_cast<const float4*>(base + (4 * DR_TB + (t >> 2)) * DK) + j);
+        if ((t & 3) == 3 || t + 1 == n) state_scale<LPC>(s, reinterpret_cast<const float4*>(base + (4 * DR_TB + (t >> 2)) * DK) + j);
       }
       if (blk + 1 == n_blk) {
         float none[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        group_sums(po, none);
+        group_sums<LPC>(j, po, none);
         store_out(orow + (int64_t)(p.S - 1) * o_ld, true);
       }
     }
     block_barrier();
   }
-  if (active) {
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-#pragma unroll
-        for (int w = 0; w < 2; ++w) {
-          const int r = i * 2 + (e >> 1);
-          const float4 v = (e & 1) ? make_float4(s[w * 4][r].y, s[w * 4 + 1][r].y, s[w * 4 + 2][r].y, s[w * 4 + 3][r].y)
-                                   : make_float4(s[w * 4][r].x, s[w * 4 + 1][r].x, s[w * 4 + 2][r].x, s[w * 4 + 3][r].x);
-          *reinterpret_cast<float4*>(srow + (int64_t)(i * LPC * 4 + e) * p.dv_pad + w * 4) = v;
-        }
-  }
+  if (active) state_store<LPC>(s, srow, p.dv_pad);
 }
 
 // ----------------------------------------------------------------------------- one token (decode)
@@ -607,17 +509,17 @@ delta_step_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
   auto fetch = [&](int column, int channel, const float* w, float (&x)[4], float (&wt)[4]) {
 #pragma unroll
     for (int k = 0; k < 4; ++k) {             // k taps back
-      x[k] = k == 0 ? dr_f<T>(row[column]) : k <= halo ? dr_f<T>(hb[(int64_t)(halo - k) * hist_ld + channel]) : 0.f;
+      x[k] = k == 0 ? rec_f<T>(row[column]) : k <= halo ? rec_f<T>(hb[(int64_t)(halo - k) * hist_ld + channel]) : 0.f;
       wt[k] = k <= halo ? w[halo - k] : 0.f;
     }
   };
   auto finish = [&](int channel, const float* w, const float (&x)[4], const float (&wt)[4]) {
     float y = fmaf(x[3], wt[3], fmaf(x[2], wt[2], fmaf(x[1], wt[1], x[0] * wt[0])));
-    for (int k = 4; k <= halo; ++k) y = fmaf(dr_f<T>(hb[(int64_t)(halo - k) * hist_ld + channel]), w[halo - k], y);
-    return y * dr_sigmoid<FAST>(y);
+    for (int k = 4; k <= halo; ++k) y = fmaf(rec_f<T>(hb[(int64_t)(halo - k) * hist_ld + channel]), w[halo - k], y);
+    return y * rec_sigmoid<FAST>(y);
   };
   float xq[4], wq[4], xk[4], wk[4], xv[4], wv[4], decay = 0.f, bias = 0.f;
-  const int cq = hk * p.dim + tid, cv = h * p.vdim + col0 + tid, ca = h * p.dim + tid;
+  const int cq = hk * p.dim + tid, cv = h * p.vdim + col0 + tid, ca = p.head_decay ? h : h * p.dim + tid;
   const bool has_v = tid < 64 && col0 + tid < p.vdim;
   if (tid < p.dim) {                          // dim <= 256
     fetch(p.q_col + cq, cq, p.conv_q + (int64_t)cq * p.taps, xq, wq);
@@ -626,7 +528,7 @@ delta_step_kernel(const T* __restrict__ proj, const T* __restrict__ hist, int64_
     bias = p.dt_bias[ca];
   }
   if (has_v) fetch(p.v_col + cv, 2 * kc + cv, p.conv_v + (int64_t)cv * p.taps, xv, wv);
-  const float beta = dr_sigmoid<FAST>(dr_f<T>(row[p.b_col + h]));
+  const float beta = rec_sigmoid<FAST>(rec_f<T>(row[p.b_col + h]));
   float q = 0.f, k = 0.f;
   if (tid < p.dim) {
     q = finish(cq, p.conv_q + (int64_t)cq * p.taps, xq, wq);
@@ -692,8 +594,8 @@ static int launch_delta_step(const void* proj, const void* hist, int64_t hist_b,
 }
 
 // ----------------------------------------------------------------------------- output gate + convolution history
-// out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate), one warp per (token, head); the blocks
-// behind them move the last taps - 1 convolution inputs of every channel into the history.
+// out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * act(gate), act = sigmoid or silu, one warp per (token, head); the
+// blocks behind them move the last taps - 1 convolution inputs of every channel into the history.
 struct DeltaOutParams {
   int B, S, H, vdim, taps;
   int channels;                 // history channels, columns conv_col .. of a projection row
@@ -701,6 +603,8 @@ struct DeltaOutParams {
   int64_t ld, ld_gate, hist_b, hist_ld;
   float eps;
   int out_blocks;
+  int gate_silu;                // the gate passes silu instead of sigmoid
+  int w_head;                   // norm weights: stride from one head's to the next (0: shared by the heads)
 };
 
 template <typename T>
@@ -721,8 +625,8 @@ delta_out_kernel(const float* __restrict__ o, const T* __restrict__ gate, const 
     ss = warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)p.vdim + p.eps);
     for (int i = lane; i < p.vdim; i += 32) {
-      const float g = dr_sigmoid<false>(dr_f<T>(gate[t * p.ld_gate + h * p.vdim + i]));
-      const float y = x[i] * inv * w[i] * g;
+      const float z = rec_f<T>(gate[t * p.ld_gate + h * p.vdim + i]), g = rec_sigmoid<false>(z);
+      const float y = x[i] * inv * w[h * p.w_head + i] * (p.gate_silu ? z * g : g);
       if (sizeof(T) == 2) reinterpret_cast<__nv_bfloat16*>(out)[item * p.vdim + i] = __float2bfloat16_rn(y);
       else reinterpret_cast<float*>(out)[item * p.vdim + i] = y;
     }
@@ -820,10 +724,13 @@ KD_API int kd_delta_rule(const kd_tensor* proj, int q_col, int k_col, int v_col,
   KD_TRY(f32_vec(conv_k, (int64_t)kv_heads * dim * p.taps, "conv_k", &p.conv_k));
   KD_TRY(f32_vec(conv_v, (int64_t)heads * vdim * p.taps, "conv_v", &p.conv_v));
   KD_TRY(f32_vec(neg_rate, heads, "neg_rate", &p.neg_rate));
-  KD_TRY(f32_vec(dt_bias, (int64_t)heads * dim, "dt_bias", &p.dt_bias));
+  // (one decay per head: a bias for every head; with key heads of one channel the two forms are the same)
+  p.head_decay = dt_bias && numel(dt_bias) == heads;
+  const int64_t decays = p.head_decay ? heads : (int64_t)heads * dim;
+  KD_TRY(f32_vec(dt_bias, decays, "dt_bias", &p.dt_bias));
   KD_TRY(kd_delta_state_shape(dim, vdim, &p.dk_pad, &p.dv_pad));
   const int64_t T = (int64_t)p.B * p.S;
-  KD_REQUIRE(decay->dtype == KD_F32 && decay->ndim == 2 && decay->strides[1] == 1 && decay->shape[0] == T && decay->shape[1] >= (int64_t)heads * dim, "decay must be fp32 [T, heads*dim]");
+  KD_REQUIRE(decay->dtype == KD_F32 && decay->ndim == 2 && decay->strides[1] == 1 && decay->shape[0] == T && decay->shape[1] >= decays, "decay must be fp32 [T, heads*dim] or [T, heads], like dt_bias");
   p.ld_a = decay->strides[0];
   KD_REQUIRE(history->ndim == 3 && history->dtype == proj->dtype && history->strides[2] == 1 && history->shape[0] >= p.B &&
                  history->shape[1] >= p.taps - 1 && history->shape[2] == C, "history must be [B, taps-1, channels] of proj's type");
@@ -853,8 +760,8 @@ KD_API int kd_delta_rule(const kd_tensor* proj, int q_col, int k_col, int v_col,
   return launch_delta_lpc<float>(pp, ph, history->strides[0], history->strides[1], p);
 }
 
-KD_API int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, float eps, const kd_tensor* proj, int conv_col, int taps,
-                        const kd_tensor* history, const kd_tensor* out) {
+KD_API int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, float eps, int gate_act, const kd_tensor* proj,
+                        int conv_col, int taps, const kd_tensor* history, const kd_tensor* out) {
   KD_TRY(require_init());
   KD_REQUIRE(o && gate && norm_weight && proj && history && out, "null tensor");
   KD_REQUIRE(proj->ndim == 3 && proj->strides[2] == 1 && proj->strides[0] == proj->strides[1] * proj->shape[1] && (proj->dtype == KD_BF16 || proj->dtype == KD_F32),
@@ -876,6 +783,8 @@ KD_API int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tens
   KD_REQUIRE(conv_col >= 0 && conv_col + p.channels <= proj->shape[2], "columns exceed the projection row");
   p.ld = proj->strides[1]; p.ld_gate = gate->strides[0]; p.hist_b = history->strides[0]; p.hist_ld = history->strides[1];
   p.eps = eps;
+  KD_REQUIRE(gate_act == KD_GATE_SIGMOID || gate_act == KD_GATE_SILU, "unknown gate activation %d", gate_act);
+  p.gate_silu = gate_act == KD_GATE_SILU;
   p.out_blocks = (int)((T * p.H + 7) / 8);
   const int hist_blocks = taps > 1 ? (int)(((int64_t)p.B * p.channels + 255) / 256) : 0;
   void *po, *pg, *pp, *ph, *pout;
@@ -889,5 +798,35 @@ KD_API int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tens
     KD_CUDA_CHECK(launch_ex(delta_out_kernel<__nv_bfloat16>, grid, dim3(256), 0, (const float*)po, (const __nv_bfloat16*)pg, w, (const __nv_bfloat16*)pp, (__nv_bfloat16*)ph, (__nv_bfloat16*)pout, p));
   else
     KD_CUDA_CHECK(launch_ex(delta_out_kernel<float>, grid, dim3(256), 0, (const float*)po, (const float*)pg, w, (const float*)pp, (float*)ph, (float*)pout, p));
+  return after_launch("delta_out_kernel");
+}
+
+KD_API int kd_gated_head_norm(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, int heads, float eps, int gate_act,
+                              const kd_tensor* out) {
+  KD_TRY(require_init());
+  KD_REQUIRE(o && gate && norm_weight && out, "null tensor");
+  KD_REQUIRE(o->dtype == KD_F32 && o->ndim == 2 && is_contiguous(o) && heads >= 1 && o->shape[1] % heads == 0 && o->shape[1] > 0, "o must be contiguous fp32 [T, heads*vdim]");
+  KD_REQUIRE(gate_act == KD_GATE_SIGMOID || gate_act == KD_GATE_SILU, "unknown gate activation %d", gate_act);
+  DeltaOutParams p{};
+  const int64_t T = o->shape[0];
+  p.B = 1; p.S = (int)T; p.H = heads; p.vdim = (int)(o->shape[1] / heads); p.taps = 1;
+  p.eps = eps;
+  p.gate_silu = gate_act == KD_GATE_SILU;
+  p.w_head = numel(norm_weight) == p.vdim ? 0 : p.vdim;
+  const float* w;
+  KD_TRY(f32_vec(norm_weight, p.w_head ? o->shape[1] : p.vdim, "norm_weight", &w));
+  KD_REQUIRE((gate->dtype == KD_BF16 || gate->dtype == KD_F32) && gate->ndim == 2 && gate->strides[1] == 1 && gate->shape[0] == T && gate->shape[1] >= o->shape[1], "gate must be [T, heads*vdim], bf16 or fp32");
+  KD_REQUIRE(out->dtype == gate->dtype && is_contiguous(out) && numel(out) == numel(o), "out must be [T, heads*vdim] of gate's type");
+  if (T == 0) return KD_OK;
+  p.ld_gate = gate->strides[0];
+  p.out_blocks = (int)((T * p.H + 7) / 8);
+  void *po, *pg, *pout;
+  KD_TRY(tensor_ptr(o, &po));
+  KD_TRY(tensor_ptr(gate, &pg));
+  KD_TRY(tensor_ptr(out, &pout));
+  if (gate->dtype == KD_BF16)
+    KD_CUDA_CHECK(launch_ex(delta_out_kernel<__nv_bfloat16>, dim3(p.out_blocks), dim3(256), 0, (const float*)po, (const __nv_bfloat16*)pg, w, (const __nv_bfloat16*)nullptr, (__nv_bfloat16*)nullptr, (__nv_bfloat16*)pout, p));
+  else
+    KD_CUDA_CHECK(launch_ex(delta_out_kernel<float>, dim3(p.out_blocks), dim3(256), 0, (const float*)po, (const float*)pg, w, (const float*)nullptr, (float*)nullptr, (float*)pout, p));
   return after_launch("delta_out_kernel");
 }

@@ -271,3 +271,27 @@ KD_API int kd_linear_ex(const kd_tensor* x, const kd_tensor* weight, const kd_te
   }
   return KD_OK;
 }
+
+KD_API int kd_linear_tanh(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* out) {
+  KD_TRY(require_init());
+  KD_REQUIRE(x && weight && out, "null tensor");
+  KD_REQUIRE(x->ndim == 2 && x->strides[1] == 1 && weight->ndim == 2 && is_contiguous(weight) && x->dtype == weight->dtype && x->dtype == out->dtype &&
+                 (x->dtype == KD_BF16 || x->dtype == KD_F32) && x->shape[1] == weight->shape[1] && out->ndim == 2 && is_contiguous(out) &&
+                 out->shape[0] == x->shape[0] && out->shape[1] == weight->shape[0],
+             "kd_linear_tanh needs x [M,K] with unit column stride, a contiguous weight [N,K] and out [M,N], one type");
+  const int64_t M = x->shape[0], K = x->shape[1], N = weight->shape[0], ldx = x->strides[0];
+  if (M == 0) return KD_OK;
+  void *px, *pw, *po;
+  KD_TRY(tensor_ptr(x, &px));
+  KD_TRY(tensor_ptr(weight, &pw));
+  KD_TRY(tensor_ptr(out, &po));
+  if (x->dtype == KD_BF16 && K % 8 == 0 && N % 8 == 0 && ldx % 8 == 0 && M < (1ll << 30) &&
+      ((reinterpret_cast<uintptr_t>(px) | reinterpret_cast<uintptr_t>(pw) | reinterpret_cast<uintptr_t>(po)) & 15) == 0)
+    return gemm_bf16_bias_act(px, ldx, pw, K, po, N, 0, nullptr, 0, (int)M, (int)N, (int)K, KD_EPI_NONE, nullptr, 2);
+  kd_matmul_cfg cfg = {};
+  cfg.M = M; cfg.N = N; cfg.K = K;
+  cfg.transpose_b = 1;
+  cfg.alpha = 1.0f;
+  KD_TRY(matmul_f32_dispatch(&cfg, x, weight, nullptr, out));
+  return kd_pointwise(KD_OP_TANH, out, nullptr, 0.f, out);
+}

@@ -89,7 +89,7 @@ struct GemmParams {
   int64_t ldr;
   int epi;
   const __nv_bfloat16* bias;   // [N] added to the accumulator before the activation and the residual, or null
-  int act;                     // 0 none, 1 GELU (tanh form) after the bias
+  int act;                     // after the bias: 0 none, 1 GELU (tanh form), 2 tanh
   int wide_store;              // bf16 output rows start on 32-byte boundaries: 32-byte vector stores
   int wide_f32, wide_resid;    // the same for an fp32 output and for the residual operand
   int num_m_tiles, num_n_tiles;
@@ -111,10 +111,11 @@ struct GemmParams {
   float* tail;
   int tail_col;
   int64_t ld_tail;
-  // grouped: A rows [group_off[g], group_off[g+1]) meet W rows [g N, (g+1) N); offsets in device memory
+  // grouped: A rows [group_off[g], group_off[g+1]) meet W rows [g N, (g+1) N); offsets in device memory, or
+  // (group_off null) group_rows rows each
   const int* group_off;
-  int groups;
-  float glu_limit;        // epi == 4: clamped GLU, see clamped_glu_f
+  int groups, group_rows;
+  float glu_limit;        // epi == 4: clamped GLU, see clamped_glu_f; epi == 5: GELU(gate) * up
 };
 
 constexpr int GEMM_MAX_GROUPS = 1024;
@@ -159,6 +160,14 @@ __device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit
   return g * r * (u + 1.0f);
 }
 
+// tanh x = 1 - 2 / (1 + exp(2 x))
+__device__ __forceinline__ float tanh_f(float x) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * (2.0f * 1.4426950408889634f)));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return fmaf(-2.0f, r, 1.0f);
+}
+
 template <int BLOCK_N, int STAGES>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b, GemmParams p) {
@@ -201,12 +210,13 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
   const int num_k_blocks = (p.K + GEMM_BK - 1) / GEMM_BK;
   int num_m_tiles = p.num_m_tiles;
   __shared__ int group_tile[GEMM_MAX_GROUPS + 1];      // first 128-row tile of every group
+  auto group_row = [&](int g) { return p.group_off ? p.group_off[g] : g * p.group_rows; };
   if (p.groups > 0) {
     if (warp == 0) {
       int carry = 0;
       for (int base = 0; base < p.groups; base += 32) {
         const int g = base + lane;
-        const int c = g < p.groups ? (p.group_off[g + 1] - p.group_off[g] + GEMM_BM - 1) / GEMM_BM : 0;
+        const int c = g < p.groups ? (group_row(g + 1) - group_row(g) + GEMM_BM - 1) / GEMM_BM : 0;
         int inc = c;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -230,8 +240,8 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
       const int mid = (lo + hi + 1) >> 1;
       if (group_tile[mid] <= m_tile) lo = mid; else hi = mid - 1;
     }
-    row0 = p.group_off[lo] + (m_tile - group_tile[lo]) * GEMM_BM;
-    row_end = p.group_off[lo + 1];
+    row0 = group_row(lo) + (m_tile - group_tile[lo]) * GEMM_BM;
+    row_end = group_row(lo + 1);
     w_row = lo * p.N;
   };
 
@@ -370,8 +380,8 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                                                             pack_bf16(__uint_as_float(x[g * 8 + 6]), __uint_as_float(x[g * 8 + 7])));
           }
         }
-      } else if (p.epi == 2 || p.epi == 4) {
-        // SiLU(gate) * up, or the clamped GLU.  Weight rows interleave 16 gate rows with the 16 matching up rows, so each
+      } else if (p.epi == 2 || p.epi == 4 || p.epi == 5) {
+        // SiLU(gate) * up, the clamped GLU, or GELU(gate) * up.  Weight rows interleave 16 gate rows with the 16 matching up rows, so each
         // 32-column chunk of the accumulator holds 16 (gate, up) pairs and yields 16 outputs.
         __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(p.out) + (int64_t)row * p.ldo + (int64_t)n_tile * (BLOCK_N / 2);
         auto process = [&](uint32_t (&r)[32], const int c0) {
@@ -383,6 +393,11 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
               for (int e = 0; e < 8; ++e)
                 o[e] = pack_bf16(clamped_glu_f(__uint_as_float(r[2 * e]), __uint_as_float(r[16 + 2 * e]), p.glu_limit),
                                  clamped_glu_f(__uint_as_float(r[2 * e + 1]), __uint_as_float(r[16 + 2 * e + 1]), p.glu_limit));
+            } else if (p.epi == 5) {
+#pragma unroll
+              for (int e = 0; e < 8; ++e)
+                o[e] = pack_bf16(gelu_f(__uint_as_float(r[2 * e])) * __uint_as_float(r[16 + 2 * e]),
+                                 gelu_f(__uint_as_float(r[2 * e + 1])) * __uint_as_float(r[16 + 2 * e + 1]));
             } else
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
@@ -450,6 +465,9 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
             if (p.act == 1) {
 #pragma unroll
               for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(gelu_f(__uint_as_float(r[i])));
+            } else if (p.act == 2) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(tanh_f(__uint_as_float(r[i])));
             }
             if (p.epi == 1) {
               if (p.out_f32) {
@@ -616,13 +634,14 @@ int gemm_bf16_bias_act(const void* A, int64_t lda, const void* W, int64_t ldw, v
   KD_REQUIRE((bias == nullptr && act == 0) || epi == 0 || epi == 1, "gemm: bias / activation combine only with the plain and residual epilogues");
   KD_REQUIRE((reinterpret_cast<uintptr_t>(bias) & 15) == 0, "gemm: bias must be 16-byte aligned");
   KD_REQUIRE(K % 8 == 0, "gemm: K=%d must be a multiple of 8 for the tensor-core path", K);
-  const int n_out = epi == 2 ? N / 2 : N;
+  const bool glu = epi == KD_EPI_SWIGLU || epi == KD_EPI_GEGLU;
+  const int n_out = glu ? N / 2 : N;
   KD_REQUIRE(n_out % 8 == 0 && ldo % (out_f32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0,
              "gemm: output width / leading dimension / address not 16-byte aligned");
   if (epi == 1)
     KD_REQUIRE(resid != nullptr && ldr % (out_f32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(resid) & 15) == 0,
                "gemm: residual operand must be 16-byte aligned");
-  if (epi == 2) KD_REQUIRE(N % 32 == 0 && !out_f32, "gemm: SwiGLU epilogue needs N %% 32 == 0 and a bf16 output");
+  if (glu) KD_REQUIRE(N % 32 == 0 && !out_f32, "gemm: the gated epilogue needs N %% 32 == 0 and a bf16 output");
   if (tail != nullptr)
     KD_REQUIRE(epi == 0 && tail_col % 32 == 0 && tail_col < N && ld_tail % 4 == 0 && (reinterpret_cast<uintptr_t>(tail) & 15) == 0,
                "gemm: the fp32 tail starts at a multiple of 32 columns (got %d of %d) and is 16-byte aligned", tail_col, N);
@@ -655,16 +674,17 @@ int gemm_bf16_bias_act(const void* A, int64_t lda, const void* W, int64_t ldw, v
 }
 
 // out[rows of g, N or N/2] = epilogue(A[rows of g, K] * W[g][N, K]^T) for all groups g (experts) in one launch.
-int gemm_bf16_grouped(const void* A, const void* W, void* out, const int* group_off, int R, int groups, int N, int K, int glu, float limit) {
+int gemm_bf16_grouped(const void* A, const void* W, void* out, const int* group_off, int R, int groups, int N, int K, int epi, float limit) {
+  const bool glu = epi != KD_EPI_NONE;
   KD_REQUIRE(R > 0 && groups > 0 && groups <= GEMM_MAX_GROUPS && K % 8 == 0, "grouped gemm: %d rows, %d groups, K=%d", R, groups, K);
   const int n_out = glu ? N / 2 : N;
   GemmParams p{};
   p.M = R; p.N = N; p.K = K;
   p.out = out; p.ldo = n_out;
-  p.epi = glu ? 4 : 0;
+  p.epi = epi;
   p.glu_limit = limit;
   p.wide_store = n_out % 16 == 0 && (reinterpret_cast<uintptr_t>(out) & 31) == 0;
-  p.group_off = group_off; p.groups = groups;
+  p.group_off = group_off; p.groups = groups; p.group_rows = R / groups;
   p.err = ctx().error_flag;
   CUtensorMap ta, tb;
   KD_TRY(make_tmap_bf16_2d(&ta, A, (uint64_t)R, (uint64_t)K, (uint64_t)K, GEMM_BM, GEMM_BK));
@@ -721,7 +741,7 @@ struct SkinnyParams {
   float* out_f32;         // [splits][Mb][N]
   int64_t ldo;            // row stride of out_bf16
   __nv_bfloat16* out_bf16;  // [Mb][N] (or [Mb][N/2] with the SiLU*up epilogue), only with splits == 1
-  int swiglu;             // rows of W interleave 16 gate / 16 up rows: write silu(gate)*up
+  int glu;                // rows of W interleave 16 gate / 16 up rows: 1 writes silu(gate)*up, 2 gelu(gate)*up
   float* tail;            // weight rows from tail_row on: fp32 [Mb][ld_tail] instead of the bf16 output
   int tail_row, ld_tail;
   float alpha;            // factor of the fp32 outputs
@@ -822,7 +842,7 @@ gemm_skinny_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
 #pragma unroll
           for (int i = 0; i < 16; ++i) r[i] = 0u;
         }
-        if (p.swiglu) {
+        if (p.glu) {
           // lanes 0-15 of a warp hold 16 gate rows, lanes 16-31 the matching up rows
           const int j = (n_tile * 128 + q * 32) / 2 + (lane & 15);
 #pragma unroll
@@ -831,7 +851,7 @@ gemm_skinny_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
             const float other = __shfl_xor_sync(0xffffffffu, mine, 16);
             const int m = c0 + i;
             if (lane < 16 && m < p.Mb && j < p.N / 2)
-              p.out_bf16[(int64_t)m * (p.N / 2) + j] = __float2bfloat16_rn(silu_f(mine) * other);
+              p.out_bf16[(int64_t)m * (p.N / 2) + j] = __float2bfloat16_rn((p.glu == 2 ? gelu_f(mine) : silu_f(mine)) * other);
           }
         } else if (n_ok) {
 #pragma unroll
@@ -871,12 +891,12 @@ int gemm_skinny_auto_splits(int N, int K) {
 // x [Mb<=128, K] bf16, W [N, K] bf16 -> fp32 partials [splits][Mb][N] (or bf16 [Mb][N] when
 // out_bf16 != NULL and splits == 1).
 int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int Mb, int N, int K, int splits,
-                     float* out_f32, void* out_bf16, int swiglu, float alpha, float* tail, int tail_row, int ld_tail) {
+                     float* out_f32, void* out_bf16, int glu, float alpha, float* tail, int tail_row, int ld_tail) {
   KD_REQUIRE(Mb >= 1 && Mb <= 128, "skinny gemm: %d rows; this path handles 1..128", Mb);
   KD_REQUIRE(N > 0 && K > 0 && K % 8 == 0, "skinny gemm: K=%d must be a positive multiple of 8", K);
   KD_REQUIRE(splits >= 1, "skinny gemm: splits must be >= 1");
   KD_REQUIRE(out_bf16 == nullptr || splits == 1, "skinny gemm: bf16 output needs splits == 1");
-  KD_REQUIRE(!swiglu || (out_bf16 != nullptr && N % 32 == 0), "skinny gemm: the SiLU*up epilogue needs a bf16 output and N %% 32 == 0");
+  KD_REQUIRE(!glu || (out_bf16 != nullptr && N % 32 == 0), "skinny gemm: the gated epilogue needs a bf16 output and N %% 32 == 0");
   SkinnyParams p{};
   p.Mb = Mb; p.N = N; p.K = K;
   p.mb_pad = (Mb + 15) / 16 * 16;
@@ -899,7 +919,7 @@ int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int
   p.tmem_cols = p.mb_pad <= 32 ? 32 : (p.mb_pad <= 64 ? 64 : 128);
   p.out_f32 = out_f32;
   p.out_bf16 = static_cast<__nv_bfloat16*>(out_bf16);
-  p.swiglu = swiglu;
+  p.glu = glu;
   p.alpha = alpha;
   p.tail = tail; p.tail_row = tail_row; p.ld_tail = ld_tail;
   p.ldo = tail ? tail_row : N;

@@ -172,29 +172,37 @@ __device__ __forceinline__ float clamped_glu_exact(float g, float u, float limit
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
 
+// gate and up of one output (epilogue: KD_EPI_SWIGLU, KD_EPI_CLAMPED_GLU or KD_EPI_GEGLU)
+__device__ __forceinline__ float glu_exact(float g, float u, int epilogue, float limit) {
+  if (epilogue == KD_EPI_CLAMPED_GLU) return clamped_glu_exact(g, u, limit);
+  if (epilogue == KD_EPI_SWIGLU) return g / (1.0f + expf(-g)) * u;
+  return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * g * g, g, g))) * u;
+}
+
 constexpr int GL_BM = 32, GL_BN = 32, GL_BK = 32;
 
 // 32 x 32 output tile, 256 threads (4 rows each); with the GLU epilogue two accumulators per output.
 template <typename T, bool GLU>
 __global__ void __launch_bounds__(256)
-moe_linear_kernel(const T* __restrict__ x, const T* __restrict__ w, const int* __restrict__ offsets, int E, int N, int K, float limit,
-                  T* __restrict__ out) {
+moe_linear_kernel(const T* __restrict__ x, const T* __restrict__ w, const int* __restrict__ offsets, int per, int E, int N, int K, int epilogue,
+                  float limit, T* __restrict__ out) {
   __shared__ float xs[GL_BM][GL_BK + 1];
   __shared__ float wg[GL_BN][GL_BK + 1];
   __shared__ float wu[GLU ? GL_BN : 1][GL_BK + 1];
   __shared__ int sel[3];
   const int n_out = GLU ? N / 2 : N;
-  // blockIdx.y enumerates the 32-row tiles of all experts
+  // blockIdx.y enumerates the 32-row tiles of all experts (without offsets every expert has `per` rows)
   if (threadIdx.x == 0) {
+    auto off = [&](int e) { return offsets ? offsets[e] : e * per; };
     int left = blockIdx.y, e = 0;
     for (; e < E; ++e) {
-      const int tiles = (offsets[e + 1] - offsets[e] + GL_BM - 1) / GL_BM;
+      const int tiles = (off(e + 1) - off(e) + GL_BM - 1) / GL_BM;
       if (left < tiles) break;
       left -= tiles;
     }
     sel[0] = e;
-    sel[1] = e < E ? offsets[e] + left * GL_BM : 0;
-    sel[2] = e < E ? offsets[e + 1] : 0;
+    sel[1] = e < E ? off(e) + left * GL_BM : 0;
+    sel[2] = e < E ? off(e + 1) : 0;
   }
   __syncthreads();
   const int e = sel[0], row0 = sel[1], row_end = sel[2];
@@ -229,14 +237,29 @@ moe_linear_kernel(const T* __restrict__ x, const T* __restrict__ w, const int* _
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int r = row0 + ty + 8 * i;
-    if (r < row_end) out[(int64_t)r * n_out + j] = (T)(GLU ? clamped_glu_exact(acc[i], acc2[i], limit) : acc[i]);
+    if (r < row_end) out[(int64_t)r * n_out + j] = (T)(GLU ? glu_exact(acc[i], acc2[i], epilogue, limit) : acc[i]);
   }
 }
 
 template <typename T>
-static void launch_moe_linear(const void* x, const void* w, const int* off, int E, int N, int K, int glu, float limit, void* out, dim3 grid) {
-  if (glu) moe_linear_kernel<T, true><<<grid, 256, 0, ctx().stream>>>((const T*)x, (const T*)w, off, E, N, K, limit, (T*)out);
-  else moe_linear_kernel<T, false><<<grid, 256, 0, ctx().stream>>>((const T*)x, (const T*)w, off, E, N, K, limit, (T*)out);
+static void launch_moe_linear(const void* x, const void* w, const int* off, int per, int E, int N, int K, int epi, float limit, void* out, dim3 grid) {
+  if (epi != KD_EPI_NONE) moe_linear_kernel<T, true><<<grid, 256, 0, ctx().stream>>>((const T*)x, (const T*)w, off, per, E, N, K, epi, limit, (T*)out);
+  else moe_linear_kernel<T, false><<<grid, 256, 0, ctx().stream>>>((const T*)x, (const T*)w, off, per, E, N, K, epi, limit, (T*)out);
+}
+
+// Rows of group e (offsets, or R / E rows each) against weight e; tensor cores where the operands allow.
+static int grouped_linear(int dtype, const void* x, const void* w, const int* off, int64_t R, int64_t E, int64_t N, int64_t K, int epi, float limit, void* out) {
+  const int64_t n_out = epi != KD_EPI_NONE ? N / 2 : N;
+  if (dtype == KD_BF16 && K % 8 == 0 && n_out % 8 == 0 && epi != KD_EPI_SWIGLU &&
+      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0)
+    return gemm_bf16_grouped(x, w, out, off, (int)R, (int)E, (int)N, (int)K, epi, limit);
+  const int64_t tiles = R / GL_BM + (E < R ? E : R) + 1;
+  KD_REQUIRE(tiles <= 65535, "grouped linear (CUDA cores): too many row tiles (%lld)", (long long)tiles);
+  dim3 grid((unsigned)((n_out + GL_BN - 1) / GL_BN), (unsigned)tiles);
+  const int per = (int)(R / E);
+  if (dtype == KD_F32) launch_moe_linear<float>(x, w, off, per, (int)E, (int)N, (int)K, epi, limit, out, grid);
+  else launch_moe_linear<__nv_bfloat16>(x, w, off, per, (int)E, (int)N, (int)K, epi, limit, out, grid);
+  return after_launch("moe_linear_kernel");
 }
 
 static int i32_ptr(const kd_tensor* t, int64_t n, const char* what, int** out) {
@@ -308,31 +331,48 @@ KD_API int kd_moe_gather(const kd_tensor* h, const kd_tensor* ids, const kd_tens
 
 KD_API int kd_moe_linear(const kd_tensor* x, const kd_tensor* weight, const kd_tensor* offsets, int epilogue, float limit, const kd_tensor* out) {
   KD_TRY(require_init());
-  KD_REQUIRE(x && weight && offsets && out, "null tensor");
-  KD_REQUIRE(epilogue == KD_EPI_NONE || epilogue == KD_EPI_CLAMPED_GLU, "kd_moe_linear: unknown epilogue %d", epilogue);
+  KD_REQUIRE(x && weight && out, "null tensor");
+  KD_REQUIRE(epilogue == KD_EPI_NONE || epilogue == KD_EPI_CLAMPED_GLU || epilogue == KD_EPI_GEGLU, "kd_moe_linear: unknown epilogue %d", epilogue);
   KD_REQUIRE(weight->ndim == 3 && is_contiguous(weight) && x->ndim == 2 && is_contiguous(x) && out->ndim == 2 && is_contiguous(out),
              "kd_moe_linear needs contiguous x [R,K], weight [E,N,K], out [R,N]");
   KD_REQUIRE(x->dtype == weight->dtype && x->dtype == out->dtype && (x->dtype == KD_BF16 || x->dtype == KD_F32), "kd_moe_linear: bf16 or fp32, one type");
   const int64_t R = x->shape[0], K = x->shape[1], E = weight->shape[0], N = weight->shape[1];
-  const bool glu = epilogue == KD_EPI_CLAMPED_GLU;
+  const bool glu = epilogue != KD_EPI_NONE;
   const int64_t n_out = glu ? N / 2 : N;
   KD_REQUIRE(weight->shape[2] == K && out->shape[0] == R && out->shape[1] == n_out, "kd_moe_linear: shapes do not match");
   KD_REQUIRE(!glu || N % 32 == 0, "the gated epilogue needs gate and up rows in blocks of 16");
   KD_REQUIRE(E >= 1 && E <= MOE_MAX_EXPERTS && R < (1ll << 30), "kd_moe_linear: %lld experts, %lld rows", (long long)E, (long long)R);
   if (R == 0) return KD_OK;
-  int* po;
-  KD_TRY(i32_ptr(offsets, E + 1, "offsets", &po));
+  int* po = nullptr;
+  if (offsets) KD_TRY(i32_ptr(offsets, E + 1, "offsets", &po));
+  else KD_REQUIRE(R % E == 0, "kd_moe_linear: %lld rows in %lld equal groups", (long long)R, (long long)E);
   void *px, *pw, *pout;
   KD_TRY(tensor_ptr(x, &px));
   KD_TRY(tensor_ptr(weight, &pw));
   KD_TRY(tensor_ptr(out, &pout));
-  if (x->dtype == KD_BF16 && K % 8 == 0 && n_out % 8 == 0 &&
-      ((reinterpret_cast<uintptr_t>(px) | reinterpret_cast<uintptr_t>(pw) | reinterpret_cast<uintptr_t>(pout)) & 15) == 0)
-    return gemm_bf16_grouped(px, pw, pout, po, (int)R, (int)E, (int)N, (int)K, glu, limit);
-  const int64_t tiles = R / GL_BM + (E < R ? E : R) + 1;
-  KD_REQUIRE(tiles <= 65535, "kd_moe_linear (CUDA cores): too many row tiles (%lld)", (long long)tiles);
-  dim3 grid((unsigned)((n_out + GL_BN - 1) / GL_BN), (unsigned)tiles);
-  if (x->dtype == KD_F32) launch_moe_linear<float>(px, pw, po, (int)E, (int)N, (int)K, glu, limit, pout, grid);
-  else launch_moe_linear<__nv_bfloat16>(px, pw, po, (int)E, (int)N, (int)K, glu, limit, pout, grid);
-  return after_launch("moe_linear_kernel");
+  return grouped_linear(x->dtype, px, pw, po, R, E, N, K, epilogue, limit, pout);
+}
+
+KD_API int kd_linear_glu(const kd_tensor* x, const kd_tensor* weight, int epilogue, const kd_tensor* out) {
+  KD_TRY(require_init());
+  KD_REQUIRE(x && weight && out, "null tensor");
+  KD_REQUIRE(epilogue == KD_EPI_SWIGLU || epilogue == KD_EPI_GEGLU, "kd_linear_glu: unknown epilogue %d", epilogue);
+  KD_REQUIRE(x->ndim == 2 && is_contiguous(x) && weight->ndim == 2 && is_contiguous(weight) && out->ndim == 2 && is_contiguous(out),
+             "kd_linear_glu needs contiguous x [M,K], weight [2I,K], out [M,I]");
+  KD_REQUIRE(x->dtype == weight->dtype && x->dtype == out->dtype && (x->dtype == KD_BF16 || x->dtype == KD_F32), "kd_linear_glu: bf16 or fp32, one type");
+  const int64_t M = x->shape[0], K = x->shape[1], N = weight->shape[0];
+  KD_REQUIRE(weight->shape[1] == K && N % 32 == 0 && out->shape[0] == M && out->shape[1] == N / 2, "kd_linear_glu: shapes do not match (gate and up rows in blocks of 16)");
+  KD_REQUIRE(M < (1ll << 30), "kd_linear_glu: %lld rows", (long long)M);
+  if (M == 0) return KD_OK;
+  void *px, *pw, *po;
+  KD_TRY(tensor_ptr(x, &px));
+  KD_TRY(tensor_ptr(weight, &pw));
+  KD_TRY(tensor_ptr(out, &po));
+  if (x->dtype == KD_BF16 && K % 8 == 0 && ((reinterpret_cast<uintptr_t>(px) | reinterpret_cast<uintptr_t>(pw) | reinterpret_cast<uintptr_t>(po)) & 15) == 0) {
+    // a handful of rows: the kernel that streams the weights, where its 128-row tiles are enough to fill the GPU
+    if (M <= 64 && N >= 128ll * (ctx().sm_count / 2))
+      return gemm_bf16_skinny(px, K, pw, K, (int)M, (int)N, (int)K, 1, nullptr, po, epilogue == KD_EPI_GEGLU ? 2 : 1);
+    return gemm_bf16(px, K, pw, K, po, N / 2, 0, nullptr, 0, (int)M, (int)N, (int)K, epilogue);
+  }
+  return grouped_linear(x->dtype, px, pw, nullptr, M, 1, N, K, epilogue, 0.f, po);
 }

@@ -1,18 +1,26 @@
-"""Engine for decoders that mix layer types: latent attention, gated delta rule, expert feed-forward,
-Dynamic Tanh norms (the Pedorax design), in bf16 or in fp32 throughout.
+"""Engine for decoders that mix layer types, in bf16 or in fp32 throughout:
+
+  Pedorax   latent attention and gated delta rule (a decay per key channel), each beside an expert feed-forward,
+            behind one Dynamic Tanh norm
+  Vogozen   sliding-window attention, WKV time mixing and gated delta rule (a decay per head), each followed by a
+            dense feed-forward, RMS norms on the sublayers' outputs
 
 One step function, `_run`, serves whole prompts, portions of prompts and decode steps: it takes S new
-tokens of B sequences at the cache's position and leaves their rows and states in the cache.  Per layer:
+tokens of B sequences at the cache's position and leaves their rows and states in the cache.  A design is a
+frame (what surrounds the sublayers: embedding, norms, residual, feed-forward, head) and a list of mixers:
 
-  one GEMM for everything that reads the norm's output (queries, latent or q/k/v, decay and gate inputs,
-  step sizes; the router's rows ride along and leave in fp32)
-  latent attention    norm + rotation + cache row -> attention over the cache rows (W_uk absorbed into the
-                      queries, W_uv applied to the combined latents), or, for long bf16 prompts, keys and
-                      values expanded once and the tcgen05 prefill kernel -> W_o
-  gated delta rule    decay / gate projections -> convolution + unit norms + recurrence in one kernel ->
-                      output norm and gate -> W_o
-  experts             route -> rows in expert order -> gate/up with the clamped GLU in the epilogue -> down
-  residual            x += mixer + weighted expert rows, and the NEXT layer's norm, in one kernel
+  frames   _ParallelFrame      h = norm(x);  x += mixer(h) + experts(h): residual and the NEXT layer's norm in one kernel
+           _SequentialFrame    x += norm(mixer(x));  x += norm(ff(x)): each residual and norm in one kernel
+  mixers   one GEMM for everything that reads the sublayer's input (small fp32 outputs such as router or decay logits
+           ride along as its tail), then
+           latent attention    norm + rotation + cache row -> attention over the cache rows (W_uk absorbed into the
+                               queries, W_uv applied to the combined latents), or, for long bf16 prompts, keys and
+                               values expanded once and the tcgen05 prefill kernel -> W_o
+           window attention    norm + rotation + cache rows -> tcgen05 prefill or split-KV decode kernel -> W_o
+           gated delta rule    convolution + unit norms + decays + recurrence in one kernel -> output norm and gate -> W_o
+           WKV                 token shift -> r, k, v, gate as one grouped GEMM, decay logits -> recurrence -> output norm
+                               and gate -> W_o
+  experts  route -> rows in expert order -> gate/up with the clamped GLU in the epilogue -> down
 
 A decode step is captured once as a CUDA graph with the position in device memory (DecoderEngine).
 
@@ -31,8 +39,10 @@ from .cache import SequenceCache
 from .core import Tensor
 from .engine import DecoderEngine, RandomInit, _r, interleave_gate_up
 from .model_utils.pedorax import ChannelDeltaSpec, ExpertsSpec, LatentAttentionSpec, PedoraxConfig
+from .model_utils.vogozen import DenseSpec, HeadDeltaSpec, VogozenConfig, WindowAttentionSpec, WkvSpec
 
-KD_EPI_NONE, KD_EPI_CLAMPED_GLU = 0, 4
+KD_EPI_NONE, KD_EPI_CLAMPED_GLU, KD_EPI_GEGLU = 0, 4, 5
+KD_GATE_SIGMOID, KD_GATE_SILU = 0, 1
 
 
 def _up(n: int, m: int) -> int:
@@ -65,6 +75,10 @@ class _Buffers:
 
 def _cols(t: Tensor, a: int, b: int) -> Tensor:
     return t.slice([slice(None)] * (t.ndim - 1) + [slice(a, b)])
+
+
+def _rows(t: Tensor, a: int, b: int) -> Tensor:
+    return t.slice([slice(a, b)] + [slice(None)] * (t.ndim - 1))
 
 
 class _Weights:
@@ -124,6 +138,17 @@ class _Weights:
     def host(self, name: str, shape) -> np.ndarray:
         return self._get(name, shape)
 
+    def padded(self, name: str, rows: int, cols: int, to_rows: int, to_cols: int) -> Tensor:
+        """A matrix with zero rows and columns behind its own."""
+        if self.random:
+            return self._draw((to_rows, to_cols))
+        a = np.zeros((to_rows, to_cols), np.float32)
+        a[:rows, :cols] = self._get(name, (rows, cols))
+        return self._put(a)
+
+    def vector_t(self, name: str, shape, random=None, plus: float = 0.0) -> Tensor:
+        return Tensor(self.vector(name, shape, random) + np.float32(plus), dtype="float32")
+
 
 class _Norm:
     def __init__(self, w: _Weights, name: str, width: int):
@@ -136,9 +161,10 @@ class _Norm:
 
 
 class _Projection:
-    """The GEMM over the norm's output: mixer columns in the engine's type, router rows in fp32 behind them."""
+    """The GEMM over a sublayer's input: columns in the engine's type, `tail` rows in fp32 behind them.
+    parts, tail: (tensor name behind the layer's prefix, rows, padded to a multiple of)."""
 
-    def __init__(self, w: _Weights, parts, width: int, prefix: str, experts: ExpertsSpec | None):
+    def __init__(self, w: _Weights, parts, width: int, prefix: str, tail=()):
         self.cols, at = {}, 0
         for key, rows, pad in parts:
             self.cols[key] = at
@@ -146,21 +172,32 @@ class _Projection:
         self.n = _up(at, 32)
         rows = [(prefix + "mix." + key, r, _up(r, pad)) for key, r, pad in parts]
         rows.append((None, 0, self.n - at))
-        self.tail = 0
-        if experts is not None:
-            self.tail = _up(experts.experts, 8)
-            rows.append((prefix + "mlp.router", experts.experts, self.tail))
+        rows += [(prefix + key, r, _up(r, pad)) for key, r, pad in tail]
+        self.tail = sum(_up(r, pad) for _, r, pad in tail)
         self.weight = w.stacked_rows(rows, width)
+
+    def __call__(self, eng: "HybridEngine", ws: _Buffers, h: Tensor, B: int, S: int):
+        """[B, S, n] in the engine's type and the tail [B*S, tail] in fp32 (or None)."""
+        T = B * S
+        out = ws("proj", (B, S, self.n), eng.dtype)
+        tail = ws("tail", (T, self.tail), "float32") if self.tail else None
+        eng.linear(h, self.weight, out.view(T, self.n), tail=tail)
+        return out, tail
+
+
+def _first(t: Tensor, B: int) -> Tensor:
+    """The first B sequences of something kept per sequence."""
+    return t if t.shape[0] == B else t.slice([slice(0, B)] + [slice(None)] * (t.ndim - 1))
 
 
 class _LatentAttention:
-    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m: LatentAttentionSpec, experts):
+    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m: LatentAttentionSpec, tail=()):
         self.m, self.i, p = m, i, f"l{i}."
         self.own = m.kvFrom is None
         parts = [("q", m.heads * (m.dim + m.rotDim), 8)]
         if self.own:
             parts.append(("dkv", m.kvRank + m.rotDim, 8))
-        self.proj = _Projection(w, parts, eng.W, p, experts)
+        self.proj = _Projection(w, parts, eng.W, p, tail)
         self.norm = Tensor(w.vector(p + "mix.dkv.norm", (m.kvRank,), 1.0), dtype="float32") if self.own else None
         self.sink = Tensor(w.vector(p + "mix.sink", (m.heads,), 0.0), dtype="float32")
         self.wo = w.matrix(p + "mix.o", (eng.W, m.heads * m.vdim))
@@ -183,11 +220,11 @@ class _LatentAttention:
                 self.wukv = w._put(np.concatenate([uk, uv], axis=0))
         self.cos, self.sin = eng.rotation(m.rotBase, m.rotDim)
 
-    def __call__(self, eng: "HybridEngine", ws: _Buffers, proj3: Tensor, B: int, S: int, pos) -> Tensor:
+    def __call__(self, eng: "HybridEngine", ws: _Buffers, h: Tensor, B: int, S: int, pos) -> Tensor:
         m, T, dt = self.m, B * S, eng.dtype
         pos_dev, pos_host = pos
-        cache = eng.cache.of(self.i).rows
-        cache = cache if cache.shape[0] == B else cache.slice([slice(0, B), slice(None), slice(None)])
+        proj3, _ = self.proj(eng, ws, h, B, S)
+        cache = _first(eng.cache.of(self.i).rows, B)
         expand = self.wukv is not None and pos_dev is None and S >= eng.expand_from
         # (the layers that read another layer's rows expand the same dense copy)
         owner = self if self.own else eng.mixers[m.kvFrom]
@@ -226,44 +263,142 @@ class _LatentAttention:
                  _r(self.sink), ctypes.c_float(m.scale), pos, _r(out))
 
 
-class _ChannelDelta:
-    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m: ChannelDeltaSpec, experts):
-        self.m, self.i, p = m, i, f"l{i}."
-        qk, vv = m.kvHeads * m.dim, m.heads * m.vdim
-        ra, rg = w.rank_of(p + "mix.a1", m.dim), w.rank_of(p + "mix.g1", m.vdim)
-        self.ra, self.rg = _up(ra, 8), _up(rg, 8)
-        # q, k, v side by side without padding: their channels are the convolution's
-        self.proj = _Projection(w, [("q", qk, 1), ("k", qk, 1), ("v", vv, 8), ("a1", ra, 8), ("g1", rg, 8), ("b", m.heads, 8)], eng.W, p, experts)
+class _DeltaRule:
+    """Gated delta rule: the parts that its forms share.  A form provides the projections, the decay logits and the gate."""
 
-        def low_rank(name, rows, rank, padded):
-            if w.random:
-                return w.matrix("", (rows, padded))
-            a = np.zeros((rows, padded), np.float32)
-            a[:, :rank] = w.host(p + name, (rows, rank))
-            return w._put(a)
-        self.wa2 = low_rank("mix.a2", m.heads * m.dim, ra, self.ra)
-        self.wg2 = low_rank("mix.g2", vv, rg, self.rg)
-        taps = lambda n, rows: Tensor(w.vector(p + f"mix.{n}.conv", (rows, m.taps), lambda s: w._rng.standard_normal(s) * 0.5), dtype="float32")  # noqa: E731
-        self.conv = taps("q", qk), taps("k", qk), taps("v", vv)
+    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m, decays: int, gate_act: int):
+        self.m, self.i, self.gate_act, p = m, i, gate_act, f"l{i}."
+        qk, vv = m.kvHeads * m.dim, m.heads * m.vdim
+        # q, k, v side by side without padding: their channels are the convolution's
+        self.parts = [("q", qk, 1), ("k", qk, 1), ("v", vv, 8)]
+        self.conv = tuple(w.vector_t(p + f"mix.{n}.conv", (rows, m.taps), lambda s: w._rng.standard_normal(s) * 0.5) for n, rows in (("q", qk), ("k", qk), ("v", vv)))
         self.neg_rate = Tensor(-np.exp(w.vector(p + "mix.A_log", (m.heads,), -1.0)), dtype="float32")
-        self.dt_bias = Tensor(w.vector(p + "mix.dt_bias", (m.heads * m.dim,), -3.0), dtype="float32")
-        self.norm = Tensor(w.vector(p + "mix.norm", (m.vdim,), 1.0), dtype="float32")
+        self.dt_bias = w.vector_t(p + "mix.dt_bias", (decays,), -3.0)
+        self.norm = w.vector_t(p + "mix.norm", (m.vdim,), 1.0)
         self.wo = w.matrix(p + "mix.o", (eng.W, vv))
 
-    def __call__(self, eng: "HybridEngine", ws: _Buffers, proj3: Tensor, B: int, S: int, pos) -> Tensor:
-        m, T, dt, c = self.m, B * S, eng.dtype, self.proj.cols
+    def __call__(self, eng: "HybridEngine", ws: _Buffers, h: Tensor, B: int, S: int, pos) -> Tensor:
+        m, T, c = self.m, B * S, self.proj.cols
         kept = eng.cache.of(self.i)
-        part = lambda t: t if t.shape[0] == B else t.slice([slice(0, B)] + [slice(None)] * (t.ndim - 1))  # noqa: E731
-        state, history = part(kept.state), part(kept.history)
-        proj2 = proj3.view(T, self.proj.n)
-        decay, gate = ws("decay", (T, m.heads * m.dim), "float32"), ws("gate", (T, m.heads * m.vdim), dt)
-        eng.linear(_cols(proj2, c["a1"], c["a1"] + self.ra), self.wa2, decay)
-        eng.linear(_cols(proj2, c["g1"], c["g1"] + self.rg), self.wg2, gate)
-        o, out = ws("delta_o", (T, m.heads * m.vdim), "float32"), ws("mixed", (T, m.heads * m.vdim), dt)
+        state, history = _first(kept.state, B), _first(kept.history, B)
+        proj3, tail = self.proj(eng, ws, h, B, S)
+        decay, gate = self.decay_and_gate(eng, ws, proj3.view(T, self.proj.n), tail)
+        o, out = ws("delta_o", (T, m.heads * m.vdim), "float32"), ws("mixed", (T, m.heads * m.vdim), eng.dtype)
         lib.call("kd_delta_rule", _r(proj3), c["q"], c["k"], c["v"], c["b"], _r(decay), m.heads, m.kvHeads, m.dim, m.vdim,
                  *(_r(t) for t in self.conv), _r(self.neg_rate), _r(self.dt_bias), _r(history), _r(state), _r(o))
-        lib.call("kd_delta_out", _r(o), _r(gate), _r(self.norm), ctypes.c_float(eng.cfg.normEps), _r(proj3), c["q"], m.taps, _r(history), _r(out))
+        lib.call("kd_delta_out", _r(o), _r(gate), _r(self.norm), ctypes.c_float(eng.cfg.normEps), self.gate_act, _r(proj3), c["q"], m.taps, _r(history), _r(out))
         return out
+
+
+class _ChannelDelta(_DeltaRule):
+    """A decay per key channel; decay and gate through low-rank factors."""
+
+    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m: ChannelDeltaSpec, tail=()):
+        super().__init__(eng, w, i, m, m.heads * m.dim, KD_GATE_SIGMOID)
+        p, vv = f"l{i}.", m.heads * m.vdim
+        ra, rg = w.rank_of(p + "mix.a1", m.dim), w.rank_of(p + "mix.g1", m.vdim)
+        self.ra, self.rg = _up(ra, 8), _up(rg, 8)
+        self.proj = _Projection(w, self.parts + [("a1", ra, 8), ("g1", rg, 8), ("b", m.heads, 8)], eng.W, p, tail)
+        self.wa2 = w.padded(p + "mix.a2", m.heads * m.dim, ra, m.heads * m.dim, self.ra)
+        self.wg2 = w.padded(p + "mix.g2", vv, rg, vv, self.rg)
+
+    def decay_and_gate(self, eng, ws, proj2: Tensor, tail):
+        m, T, c = self.m, proj2.shape[0], self.proj.cols
+        decay, gate = ws("decay", (T, m.heads * m.dim), "float32"), ws("gate", (T, m.heads * m.vdim), eng.dtype)
+        eng.linear(_cols(proj2, c["a1"], c["a1"] + self.ra), self.wa2, decay)
+        eng.linear(_cols(proj2, c["g1"], c["g1"] + self.rg), self.wg2, gate)
+        return decay, gate
+
+
+class _HeadDelta(_DeltaRule):
+    """One decay per head, whose logits leave the first GEMM in fp32; a full-rank gate through silu."""
+
+    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m: HeadDeltaSpec, tail=()):
+        super().__init__(eng, w, i, m, m.heads, KD_GATE_SILU)
+        self.proj = _Projection(w, self.parts + [("g", m.heads * m.vdim, 8), ("b", m.heads, 8)], eng.W, f"l{i}.", [("mix.a", m.heads, 8), *tail])
+
+    def decay_and_gate(self, eng, ws, proj2: Tensor, tail):
+        g, vv = self.proj.cols["g"], self.m.heads * self.m.vdim
+        return _cols(tail, 0, self.m.heads), _cols(proj2, g, g + vv)
+
+
+class _WindowAttention:
+    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m: WindowAttentionSpec, tail=()):
+        self.m, self.i, p = m, i, f"l{i}."
+        self.own = m.kvFrom is None
+        qd, vd = ctypes.c_int(0), ctypes.c_int(0)
+        lib.call("kd_attention_head_sizes", lib.DTYPES[eng.dtype][0], m.dim, m.vdim, ctypes.byref(qd), ctypes.byref(vd))
+        self.q_size, self.v_size = qd.value, vd.value
+        parts = [("q", m.heads * m.dim, 8)]
+        if self.own:
+            parts += [("k", m.kvHeads * m.dim, 8), ("v", m.kvHeads * m.vdim, 8)]
+        self.proj = _Projection(w, parts, eng.W, p, tail)
+        self.q_norm = w.vector_t(p + "mix.q.norm", (m.heads * m.dim,), 1.0)
+        self.k_norm = w.vector_t(p + "mix.k.norm", (m.kvHeads * m.dim,), 1.0) if self.own else None
+        self.sink = core.zeros((m.heads,), "float32")     # the one in the softmax denominator: a score of 0
+        self.cos, self.sin = eng.rotation(m.rotBase, m.rotDims)
+        if w.random or self.v_size == m.vdim:
+            self.wo = w.matrix(p + "mix.o", (eng.W, m.heads * self.v_size))
+        else:                                             # the padding columns of a head's output meet zeros
+            wo = np.zeros((eng.W, m.heads, self.v_size), np.float32)
+            wo[:, :, :m.vdim] = w.host(p + "mix.o", (eng.W, m.heads * m.vdim)).reshape(eng.W, m.heads, m.vdim)
+            self.wo = w._put(wo.reshape(eng.W, m.heads * self.v_size))
+
+    def __call__(self, eng: "HybridEngine", ws: _Buffers, h: Tensor, B: int, S: int, pos) -> Tensor:
+        m, c = self.m, self.proj.cols
+        pos_dev, pos_host = pos
+        proj3, _ = self.proj(eng, ws, h, B, S)
+        kept = eng.cache.of(self.i)
+        keys, values = _first(kept.keys, B), _first(kept.values, B)
+        q = ws("q", (B, S, m.heads, self.q_size), eng.dtype)
+        out = ws("mixed", (B * S, m.heads * self.v_size), eng.dtype)
+        lib.call("kd_qk_norm_rope_cache", _r(proj3), c["q"], c.get("k", -1), c.get("v", -1), m.dim, m.vdim, m.rotDims, _r(self.q_norm), _r(self.k_norm),
+                 ctypes.c_float(eng.cfg.normEps), _r(self.cos), _r(self.sin), _r(keys), _r(values), _r(pos_dev), pos_host, _r(q))
+        lib.call("kd_window_attention", _r(q), _r(keys), _r(values), _r(self.sink), ctypes.c_float(m.scale), m.window, _r(pos_dev), pos_host, _r(out))
+        return out
+
+
+class _Wkv:
+    MIXES = "rkvgw"          # order of the shifted inputs: the first four meet one matrix each in one grouped GEMM
+
+    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, m: WkvSpec, tail=()):
+        if tail:
+            raise ValueError("a WKV layer has no common projection for other rows to join")
+        self.m, self.i, p = m, i, f"l{i}."
+        n, W = m.heads * m.dim, eng.W
+        self.mu = Tensor(np.stack([w.vector(f"{p}mix.mu.{x}", (W,), 0.5) for x in self.MIXES]), dtype="float32")
+        if w.random:
+            self.w4 = w.matrix("", (4, n, W))
+        else:
+            self.w4 = w._put(np.stack([w.host(f"{p}mix.{x}", (n, W)) for x in self.MIXES[:4]]))
+        rank = w.rank_of(p + "mix.w1", 64)
+        self.rank = _up(rank, 8)
+        self.w1 = w.padded(p + "mix.w1", rank, W, self.rank, W)
+        self.w2 = w.padded(p + "mix.w2", n, rank, n, self.rank)
+        self.w0 = w.vector_t(p + "mix.w0", (n,), -1.0)
+        self.u = w.vector_t(p + "mix.u", (m.heads, m.dim), 0.5).view(n)
+        self.norm = w.vector_t(p + "mix.norm", (n,), 1.0)
+        self.wo = w.matrix(p + "mix.o", (W, n))
+
+    def __call__(self, eng: "HybridEngine", ws: _Buffers, h: Tensor, B: int, S: int, pos) -> Tensor:
+        m, T, dt, W = self.m, B * S, eng.dtype, eng.W
+        n = m.heads * m.dim
+        kept = eng.cache.of(self.i)
+        state, last = _first(kept.state, B), _first(kept.last, B)
+        mixes, rkvg = ws("mixes", (5 * T, W), dt), ws("rkvg", (4 * T, n), dt)
+        lib.call("kd_token_shift", _r(h.view(B, S, W)), _r(self.mu), _r(last), _r(mixes))
+        lib.call("kd_moe_linear", _r(_rows(mixes, 0, 4 * T)), _r(self.w4), None, KD_EPI_NONE, ctypes.c_float(0.0), _r(rkvg))
+        low, logits = ws("wkv_low", (T, self.rank), dt), ws("decay", (T, n), "float32")
+        lib.call("kd_linear_tanh", _r(_rows(mixes, 4 * T, 5 * T)), _r(self.w1), _r(low))
+        eng.linear(low, self.w2, logits)
+        r, k, v = (_rows(rkvg, x * T, (x + 1) * T).view(B, S, n) for x in range(3))
+        o, out = ws("delta_o", (T, n), "float32"), ws("mixed", (T, n), dt)
+        lib.call("kd_wkv", _r(r), _r(k), _r(v), _r(logits), _r(self.w0), _r(self.u), _r(state), _r(o))
+        lib.call("kd_gated_head_norm", _r(o), _r(_rows(rkvg, 3 * T, 4 * T)), _r(self.norm), m.heads, ctypes.c_float(eng.cfg.normEps), KD_GATE_SILU, _r(out))
+        return out
+
+
+_MIXERS = {LatentAttentionSpec: _LatentAttention, ChannelDeltaSpec: _ChannelDelta, HeadDeltaSpec: _HeadDelta, WindowAttentionSpec: _WindowAttention, WkvSpec: _Wkv}
 
 
 class _Experts:
@@ -296,8 +431,101 @@ class _Experts:
         return y, slots, weights
 
 
+class _GatedDense:
+    """Dense feed-forward, GELU(gate) * up in the GEMM's epilogue."""
+
+    def __init__(self, eng: "HybridEngine", w: _Weights, i: int, d: DenseSpec):
+        p, self.ff = f"l{i}.mlp.", _up(d.ff, 16)      # gate and up rows interleave in blocks of 16; padding is zero
+        if w.random:
+            self.wgu = w.matrix("", (2 * self.ff, eng.W))
+        else:
+            grown = lambda n: np.concatenate([w.host(p + n, (d.ff, eng.W)), np.zeros((self.ff - d.ff, eng.W), np.float32)])  # noqa: E731
+            self.wgu = w._put(interleave_gate_up(grown("gate"), grown("up")))
+        self.wdown = w.padded(p + "down", eng.W, d.ff, eng.W, self.ff)
+
+    def __call__(self, eng: "HybridEngine", ws: _Buffers, h: Tensor) -> Tensor:
+        act = ws("act", (h.shape[0], self.ff), eng.dtype)
+        lib.call("kd_linear_glu", _r(h), _r(self.wgu), KD_EPI_GEGLU, _r(act))
+        return act
+
+
+class _ParallelFrame:
+    """Pedorax: one Dynamic Tanh norm per layer feeds the mixer and, beside it, the experts."""
+
+    def __init__(self, eng: "HybridEngine", w: _Weights, cfg: PedoraxConfig):
+        self.embed = w.matrix("embed", (eng.V, eng.W))
+        self.norms, self.mixers, self.experts = [], [], []
+        for i, layer in enumerate(cfg.layers):
+            self.norms.append(_Norm(w, f"l{i}.norm1", eng.W))
+            tail = [("mlp.router", layer.experts.experts, 8)] if layer.experts is not None else []
+            self.mixers.append(_MIXERS[type(layer.mixer)](eng, w, i, layer.mixer, tail))
+            self.experts.append(_Experts(eng, w, i, layer.experts) if layer.experts is not None else None)
+        self.norms.append(_Norm(w, "final.norm", eng.W))
+        self.max_experts = max([e.e.experts for e in self.experts if e is not None], default=1)
+        self.head, self.embed_scale, self.logit_scale = self.embed, cfg.embeddingScale, cfg.logitScale
+
+    def run(self, eng: "HybridEngine", ws: _Buffers, ids: Tensor, B: int, S: int, pos) -> Tensor:
+        T, dt = B * S, eng.dtype
+        x, h = ws("x", (T, eng.W), "float32"), ws("h", (T, eng.W), dt)
+        counts = ws("moe_counts", (len(self.experts), self.max_experts), "int32")
+        lib.call("kd_fill", _r(counts), ctypes.c_double(0.0))
+        lib.call("kd_embed_dynamic_tanh", _r(self.embed), _r(ids), ctypes.c_float(self.embed_scale), *self.norms[0].args(), _r(x), _r(h))
+        for i, (mixer, experts) in enumerate(zip(self.mixers, self.experts)):
+            mixed = mixer(eng, ws, h, B, S, pos)
+            mix = self._out_projection(eng, ws, mixed, mixer.wo, x, T)
+            y = slots = weights = None
+            if experts is not None:
+                y, slots, weights = experts(eng, ws, h, ws("tail", (T, mixer.proj.tail), "float32"),
+                                            counts.slice([slice(i, i + 1), slice(0, experts.e.experts)]))
+            lib.call("kd_residual_dynamic_tanh", _r(x), _r(mix), _r(y), _r(slots), _r(weights), *self.norms[i + 1].args(), _r(x), _r(h))
+            eng.traced(x)
+        return h
+
+    @staticmethod
+    def _out_projection(eng: "HybridEngine", ws: _Buffers, mixed: Tensor, wo: Tensor, x: Tensor, T: int):
+        """x += mixed W_o^T in the GEMM's epilogue for many rows (returns None); for a few rows fp32 partial sums that
+        the residual kernel adds."""
+        if eng.dtype == "bfloat16" and T > 64 and mixed.shape[1] % 8 == 0 and eng.W % 8 == 0:
+            eng.linear(mixed, wo, x, residual=x)
+            return None
+        return eng.partial_sums(ws, mixed, wo, "float32")
+
+
+class _SequentialFrame:
+    """Vogozen: mixer, then feed-forward; each reads the residual itself and is normed before it is added."""
+
+    def __init__(self, eng: "HybridEngine", w: _Weights, cfg: VogozenConfig):
+        self.embed = w.matrix("embed", (eng.V, eng.W))
+        self.mixers, self.dense, self.norms = [], [], []
+        for i, layer in enumerate(cfg.layers):
+            self.mixers.append(_MIXERS[type(layer.mixer)](eng, w, i, layer.mixer))
+            self.dense.append(_GatedDense(eng, w, i, layer.dense) if layer.dense is not None else None)
+            # norm weights are stored around zero
+            norm = lambda n: w.vector_t(f"l{i}.{n}", (eng.W,), 0.0, plus=1.0)  # noqa: E731
+            self.norms.append((norm("norm1"), norm("norm2") if layer.dense is not None else None))
+        self.final = w.vector_t("final.norm", (eng.W,), 0.0, plus=1.0)
+        self.head, self.logit_scale = w.matrix("head", (eng.V, eng.W)), 1.0
+
+    def run(self, eng: "HybridEngine", ws: _Buffers, ids: Tensor, B: int, S: int, pos) -> Tensor:
+        T, eps, n = B * S, ctypes.c_float(eng.cfg.normEps), len(self.mixers)
+        x, h = ws("x", (T, eng.W), "float32"), ws("h", (T, eng.W), eng.dtype)
+        lib.call("kd_embed_rows", _r(self.embed), _r(ids), _r(x), _r(h))
+        for i, (mixer, dense, (norm1, norm2)) in enumerate(zip(self.mixers, self.dense, self.norms)):
+            last = i + 1 == n
+            y = eng.partial_sums(ws, mixer(eng, ws, h, B, S, pos), mixer.wo, eng.dtype)
+            lib.call("kd_residual_post_norm", _r(x), _r(y), _r(norm1), eps, _r(self.final) if last and dense is None else None, _r(x), _r(h))
+            if dense is not None:
+                y = eng.partial_sums(ws, dense(eng, ws, h), dense.wdown, eng.dtype)
+                lib.call("kd_residual_post_norm", _r(x), _r(y), _r(norm2), eps, _r(self.final) if last else None, _r(x), _r(h))
+            eng.traced(x)
+        return h
+
+
+_FRAMES = {PedoraxConfig: _ParallelFrame, VogozenConfig: _SequentialFrame}
+
+
 class HybridEngine(DecoderEngine):
-    def __init__(self, cfg: PedoraxConfig, weights, max_batch: int, max_seq_len: int):
+    def __init__(self, cfg: PedoraxConfig | VogozenConfig, weights, max_batch: int, max_seq_len: int):
         """weights: a mapping of the checkpoint's tensor names to float32 arrays (io.SafetensorStateDict, a
         dict), or a RandomInit.  cfg.dtype is "bfloat16" or "float32"."""
         cfg.validate()
@@ -306,18 +534,10 @@ class HybridEngine(DecoderEngine):
         self._init_decoding(max_batch, max_seq_len)
         self.cfg, self.dtype, self.W, self.V = cfg, cfg.dtype, cfg.hiddenSize, cfg.vocabSize
         self._tables = {}
-        w = _Weights(weights, self.dtype)
-        self.embed = w.matrix("embed", (self.V, self.W))
-        self.norms, self.mixers, self.experts = [], [], []
-        for i, layer in enumerate(cfg.layers):
-            self.norms.append(_Norm(w, f"l{i}.norm1", self.W))
-            kind = _LatentAttention if isinstance(layer.mixer, LatentAttentionSpec) else _ChannelDelta
-            self.mixers.append(kind(self, w, i, layer.mixer, layer.experts))
-            self.experts.append(_Experts(self, w, i, layer.experts) if layer.experts is not None else None)
-        self.norms.append(_Norm(w, "final.norm", self.W))
-        self.max_experts = max([e.e.experts for e in self.experts if e is not None], default=1)
-        self.cache = SequenceCache(cfg.layers, max_batch, max_seq_len, self.dtype)
-        self.expand_from = 64      # portions of at least this many tokens expand keys and values
+        self.frame = _FRAMES[type(cfg)](self, _Weights(weights, self.dtype), cfg)
+        self.mixers = self.frame.mixers
+        self.cache = SequenceCache(cfg.layers, max_batch, max_seq_len, self.dtype, self.W)
+        self.expand_from = 64      # portions of at least this many tokens expand keys and values (latent attention)
         self._prompt = _Buffers()
         self.cur_B = 0
         self.trace = None          # a list: receives the residual stream [T, W] after every layer (tests)
@@ -335,52 +555,36 @@ class HybridEngine(DecoderEngine):
     def linear(self, x: Tensor, w: Tensor, out: Tensor, residual: Tensor | None = None, alpha: float = 1.0, tail: Tensor | None = None) -> None:
         lib.call("kd_linear_ex", _r(x), _r(w), _r(residual), ctypes.c_float(alpha), _r(out), _r(tail))
 
+    def partial_sums(self, ws: _Buffers, x: Tensor, w: Tensor, dtype: str) -> Tensor:
+        """x w^T for a kernel that adds up split-K partial sums: fp32 [splits, T, W] for a few bf16 rows, else [1, T, W]
+        in `dtype`."""
+        T, k = x.shape
+        if self.dtype == "bfloat16" and T <= 64 and k % 8 == 0:
+            s = ctypes.c_int(0)
+            lib.call("kd_linear_bf16_skinny_splits", ctypes.c_int64(self.W), ctypes.c_int64(k), ctypes.byref(s))
+            y = ws("mix", (s.value, T, self.W), "float32")
+            lib.call("kd_linear_bf16_skinny", _r(x), _r(w), 0, _r(y))
+            return y
+        y = ws("mix" if dtype == "float32" else "mix16", (1, T, self.W), dtype)
+        self.linear(x, w, y.view(T, self.W))
+        return y
+
+    def traced(self, x: Tensor) -> None:
+        if self.trace is not None:
+            self.trace.append(x.dataAsync().copy())
+
     # ------------------------------------------------------------------ one step over S tokens of B sequences
     def _run(self, ws: _Buffers, ids: Tensor, B: int, S: int, pos_dev: Tensor | None, pos_host: int) -> Tensor:
         """ids: device int32/int64 [B*S].  Runs them at the given position; returns the final norm's output [B*S, W]."""
-        T, dt, c = B * S, self.dtype, self.cfg
-        x, h = ws("x", (T, self.W), "float32"), ws("h", (T, self.W), dt)
-        counts = ws("moe_counts", (len(self.experts), self.max_experts), "int32")
-        lib.call("kd_fill", _r(counts), ctypes.c_double(0.0))
-        lib.call("kd_embed_dynamic_tanh", _r(self.embed), _r(ids), ctypes.c_float(c.embeddingScale), *self.norms[0].args(), _r(x), _r(h))
-        for i, (mixer, experts) in enumerate(zip(self.mixers, self.experts)):
-            p = mixer.proj
-            proj3 = ws("proj", (B, S, p.n), dt)
-            tail = ws("tail", (T, p.tail), "float32") if p.tail else None
-            self.linear(h, p.weight, proj3.view(T, p.n), tail=tail)
-            mixed = mixer(self, ws, proj3, B, S, (pos_dev, pos_host))
-            mix = self._out_projection(ws, mixed, mixer.wo, x, T)
-            y = slots = weights = None
-            if experts is not None:
-                y, slots, weights = experts(self, ws, h, tail, counts.slice([slice(i, i + 1), slice(0, experts.e.experts)]))
-            lib.call("kd_residual_dynamic_tanh", _r(x), _r(mix), _r(y), _r(slots), _r(weights), *self.norms[i + 1].args(), _r(x), _r(h))
-            if self.trace is not None:
-                self.trace.append(x.dataAsync().copy())
-        return h
-
-    def _out_projection(self, ws: _Buffers, mixed: Tensor, wo: Tensor, x: Tensor, T: int):
-        """x += mixed W_o^T in the GEMM's epilogue for many rows (returns None); for a few rows fp32 partial sums that
-        the residual kernel adds."""
-        if self.dtype == "bfloat16" and T > 64 and mixed.shape[1] % 8 == 0 and self.W % 8 == 0:
-            self.linear(mixed, wo, x, residual=x)
-            return None
-        if self.dtype == "bfloat16" and T <= 64 and mixed.shape[1] % 8 == 0:
-            s = ctypes.c_int(0)
-            lib.call("kd_linear_bf16_skinny_splits", ctypes.c_int64(self.W), ctypes.c_int64(mixed.shape[1]), ctypes.byref(s))
-            mix = ws("mix", (s.value, T, self.W), "float32")
-            lib.call("kd_linear_bf16_skinny", _r(mixed), _r(wo), 0, _r(mix))
-            return mix
-        mix = ws("mix", (1, T, self.W), "float32")
-        self.linear(mixed, wo, mix.view(T, self.W))
-        return mix
+        return self.frame.run(self, ws, ids, B, S, (pos_dev, pos_host))
 
     def _logits(self, ws: _Buffers, rows: Tensor, out: Tensor) -> None:
-        """out [n, V] fp32 = logit_scale * rows [n, W] embed^T (64 rows a call: the vocabulary matrix streams once each)."""
+        """out [n, V] fp32 = logit_scale * rows [n, W] head^T (64 rows a call: the vocabulary matrix streams once each)."""
         n = rows.shape[0]
         for a in range(0, n, 64):
             b = min(n, a + 64)
             r, o = (t.slice([slice(a, b), slice(None)]) for t in (rows, out))
-            self.linear(r, self.embed, o, alpha=self.cfg.logitScale)
+            self.linear(r, self.frame.head, o, alpha=self.frame.logit_scale)
 
     # ------------------------------------------------------------------ prompts and portions
     def reset(self) -> None:

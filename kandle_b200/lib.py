@@ -192,7 +192,17 @@ _SIGNATURES = {
     "kd_latent_prefill": [_T] + [ctypes.c_int] * 4 + [_T, ctypes.c_int, _T, ctypes.c_int, _T, ctypes.c_float, ctypes.c_int, _T],
     "kd_delta_rule": [_T] + [ctypes.c_int] * 4 + [_T] + [ctypes.c_int] * 4 + [_T] * 8,
     "kd_delta_state_shape": [ctypes.c_int, ctypes.c_int, ctypes.POINTER(ctypes.c_int), ctypes.POINTER(ctypes.c_int)],
-    "kd_delta_out": [_T, _T, _T, ctypes.c_float, _T, ctypes.c_int, ctypes.c_int, _T, _T],
+    "kd_delta_out": [_T, _T, _T, ctypes.c_float, ctypes.c_int, _T, ctypes.c_int, ctypes.c_int, _T, _T],
+    "kd_gated_head_norm": [_T, _T, _T, ctypes.c_int, ctypes.c_float, ctypes.c_int, _T],
+    "kd_token_shift": [_T] * 4,
+    "kd_wkv": [_T] * 8,
+    "kd_linear_glu": [_T, _T, ctypes.c_int, _T],
+    "kd_linear_tanh": [_T] * 3,
+    "kd_embed_rows": [_T] * 4,
+    "kd_residual_post_norm": [_T, _T, _T, ctypes.c_float, _T, _T, _T],
+    "kd_attention_head_sizes": [ctypes.c_int] * 3 + [ctypes.POINTER(ctypes.c_int)] * 2,
+    "kd_qk_norm_rope_cache": [_T] + [ctypes.c_int] * 6 + [_T, _T, ctypes.c_float, _T, _T, _T, _T, _T, ctypes.c_int, _T],
+    "kd_window_attention": [_T] * 4 + [ctypes.c_float, ctypes.c_int, _T, ctypes.c_int, _T],
 }
 
 

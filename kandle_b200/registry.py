@@ -70,6 +70,11 @@ def _pedorax_config(c: dict, dtype: str):
     return PedoraxConfig.fromDict(c, dtype)
 
 
+def _vogozen_config(c: dict, dtype: str):
+    from .model_utils.vogozen import VogozenConfig
+    return VogozenConfig.fromDict(c, dtype)
+
+
 def _hybrid_engine(cfg, weights, max_batch, max_seq_len):
     from .hybrid_engine import HybridEngine
     return HybridEngine(cfg, weights, max_batch, max_seq_len)
@@ -77,3 +82,4 @@ def _hybrid_engine(cfg, weights, max_batch, max_seq_len):
 
 register("Qwen3ForCausalLM", ModelEntry(_qwen3_config, _qwen3_engine, ("bfloat16",)))
 register("Pedorax", ModelEntry(_pedorax_config, _hybrid_engine, ("bfloat16", "float32")))
+register("Vogozen", ModelEntry(_vogozen_config, _hybrid_engine, ("bfloat16", "float32")))

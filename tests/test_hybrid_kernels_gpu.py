@@ -260,7 +260,7 @@ def _delta_case(B, S, H, Hk, dim, vdim, taps, dtype, cuts, a_mean=-2.0, a_sd=1.0
         o, y = core.full((B * n_tok, vv), float("nan")), core.full((B * n_tok, vv), float("nan"), dtype)
         lib.call("kd_delta_rule", _r(pd), 0, qk, 2 * qk, 2 * qk + vv, _r(_put(a[:, at:at + n_tok].reshape(B * n_tok, -1))), H, Hk, dim, vdim, *(_r(x) for x in ws),
                  _r(_put(-rate)), _r(_put(bias)), _r(hist), _r(state), _r(o))
-        lib.call("kd_delta_out", _r(o), _r(_put(gate[:, at:at + n_tok].reshape(B * n_tok, -1), dtype)), _r(_put(norm_w)), F(1e-5), _r(pd), 0, taps, _r(hist), _r(y))
+        lib.call("kd_delta_out", _r(o), _r(_put(gate[:, at:at + n_tok].reshape(B * n_tok, -1), dtype)), _r(_put(norm_w)), F(1e-5), 0, _r(pd), 0, taps, _r(hist), _r(y))
         outs.append(_get(o).reshape(B, n_tok, H, vdim))
         finals.append(_get(y).reshape(B, n_tok, H, vdim))
         at += n_tok
