@@ -1,7 +1,7 @@
 """Headline benchmark: Qwen3-0.6B-architecture bf16 prefill + greedy decode, tokens/s.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--no-extras]
-    python bench.py --hybrid [--hybrid-sizes 1k,2k,4k]     (the Pedorax design beside Qwen3 at equal size)
+    python bench.py --hybrid [--hybrid-design pedorax|vogozen] [--hybrid-sizes 1k,2k,4k]     (a hybrid design beside Qwen3 at equal size)
 
 Headline workload (`config.workload` = "qwen3-0.6b-bf16-b32-p2048-d256"): random-init weights
 N(0, 0.02) of the Qwen3-0.6B architecture (28 layers, hidden 1024, 16 q / 8 kv heads x 128, MLP 3072,
@@ -75,7 +75,8 @@ def parse_args():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extras", action="store_true", help="headline only (no weak_dp / tp_4b / whisper_c5 records)")
     ap.add_argument("--extras", default="weak_dp,tp_4b,whisper_c5")
-    ap.add_argument("--hybrid", action="store_true", help="instead of the headline: the Pedorax design beside Qwen3 at equal size, one JSON line a size")
+    ap.add_argument("--hybrid", action="store_true", help="instead of the headline: a hybrid design beside Qwen3 at equal size, one JSON line a size")
+    ap.add_argument("--hybrid-design", default="pedorax", choices=["pedorax", "vogozen"])
     ap.add_argument("--hybrid-sizes", default="1k,2k,4k")
     ap.add_argument("--hybrid-layers", type=int, default=4)
     ap.add_argument("--hybrid-batch", type=int, default=32)
@@ -825,8 +826,8 @@ def main():
         import kandle_b200
         from kandle_b200 import hybrid_bench
         kandle_b200.init(0)
-        hybrid_bench.main([s for s in a.hybrid_sizes.split(",") if s], a.hybrid_layers, a.hybrid_batch, a.hybrid_prompt, a.hybrid_steps,
-                          load_peaks()[0][0])
+        hybrid_bench.main(a.hybrid_design, [s for s in a.hybrid_sizes.split(",") if s], a.hybrid_layers, a.hybrid_batch, a.hybrid_prompt, a.hybrid_steps,
+                          load_peaks()[0][0], load_peaks()[1][0])
     elif a.impl == "reference":
         run_reference(a)
     else:

@@ -1,11 +1,14 @@
-"""Small random models of the Pedorax design for the tests: configurations, weights (rounded to bf16, so that
-both sides see the same numbers) and comparisons with the plain implementation in oracle/hybrid.py."""
+"""Small random models of the hybrid designs (Pedorax here, Vogozen in vogozen_cases.py) for the tests:
+configurations, weights (rounded to bf16, so that both sides see the same numbers) and comparisons with the plain
+implementations in oracle/hybrid.py and oracle/vogozen.py."""
 from __future__ import annotations
 
 import numpy as np
 
-from kandle_b200 import lib
-from oracle import hybrid
+from kandle_b200 import lib, registry
+from oracle import hybrid, vogozen
+
+ORACLES = {"Pedorax": hybrid, "Vogozen": vogozen}
 
 
 def latent(heads=3, dim=24, rot=16, vdim=40, rank=48, scale=0.2, base=5000.0, kv_from=None):
@@ -92,9 +95,8 @@ def weights(cfg, seed=0, sharp=1.0):
 
 
 def engine(cfg, w, batch=1, max_s=256, dtype="float32"):
-    from kandle_b200.hybrid_engine import HybridEngine
-    from kandle_b200.model_utils.pedorax import PedoraxConfig
-    return HybridEngine(PedoraxConfig.fromDict(cfg, dtype), w, batch, max_s)
+    entry = registry.lookup(cfg)
+    return entry.engine(entry.config(cfg, dtype), w, batch, max_s)
 
 
 def tokens(cfg, *shape, seed=1):
@@ -114,7 +116,7 @@ def run_cut(eng, ids, cuts):
 
 
 def reference(cfg, w, ids):
-    return np.stack([hybrid.forward(cfg, w, row) for row in ids])
+    return np.stack([ORACLES[cfg["architecture"]].forward(cfg, w, row) for row in ids])
 
 
 def row_errors(got, ref):
