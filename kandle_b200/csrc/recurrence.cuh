@@ -57,11 +57,16 @@ template <> struct Raw4<__nv_bfloat16> {
     v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
     v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
   }
+  __device__ __forceinline__ void set(const float (&v)[4]) {      // of values that bf16 holds exactly
+    u.x = (__float_as_uint(v[0]) >> 16) | (__float_as_uint(v[1]) & 0xffff0000u);
+    u.y = (__float_as_uint(v[2]) >> 16) | (__float_as_uint(v[3]) & 0xffff0000u);
+  }
 };
 template <> struct Raw4<float> {
   float4 f;
   __device__ __forceinline__ void load(const float* p) { f = *reinterpret_cast<const float4*>(p); }
   __device__ __forceinline__ void get(float (&v)[4]) const { v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+  __device__ __forceinline__ void set(const float (&v)[4]) { f = make_float4(v[0], v[1], v[2], v[3]); }
 };
 
 // Rows of this lane's 8 columns; src points at (row 4 j, first column), null: zeros.

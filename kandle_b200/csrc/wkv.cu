@@ -10,6 +10,8 @@
 // by the product P of the decays so far (r P to read, k / P to write), so a token costs two packed operations per
 // pair of state entries and the group one more; a decay below 1e-6 is applied to the state at that token, between
 // its read and its write.  Two tokens' outputs are summed over a group's lanes together.
+// Eight consumer warps (208 registers a thread) and four helper warps (88); a helper warp prepares four tokens of a
+// head in as many lanes as the head has quads of channels, so a warp takes two groups of tokens of a 64-channel head.
 // Bound: fp32 pipe in prefill (2.25 dim^2 multiply-adds per head and token), HBM in decode (the state is read and
 // written once per token: 8 dim^2 bytes per head and sequence).
 #include "common.cuh"
@@ -123,13 +125,17 @@ template <int LPC> constexpr int wkv_tokens() { return LPC <= 4 ? 8 : 16; }
 // four tokens [TB/4][dk], v [TB][dv], bonus factors and flags [TB].
 __host__ __device__ constexpr int wkv_unit_floats(int tb, int dk, int dv) { return tb * (3 * dk + dv) + (tb / 4) * dk + 2 * tb; }
 
+constexpr int WKV_HELPERS = 4, WKV_THREADS = (REC_CONSUMERS + WKV_HELPERS) * 32;
+
 template <typename T, int LPC>
-__global__ void __launch_bounds__(REC_THREADS, 1)
+__global__ void __launch_bounds__(WKV_THREADS, 1)
 wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __restrict__ v_in, WkvParams p) {
   constexpr bool FAST = sizeof(T) == 2;
   constexpr int TB = wkv_tokens<LPC>();
   constexpr int DK = 16 * LPC;                 // padded key channels
   constexpr int CH = DK > 128 ? DK / 128 : 1;  // helper passes over the key channels
+  constexpr int LANES = DK < 128 ? DK / 4 : 32;                          // helper lanes that share a token's channels
+  constexpr int GPI = 32 / LANES < TB / 4 ? 32 / LANES : TB / 4;         // groups of four tokens a helper warp takes at once
   constexpr int CPW = 8 * (32 / LPC);          // columns per warp
   extern __shared__ __align__(16) float sm[];
   const int dvc = p.wpc * CPW;                 // columns of a head in this CTA
@@ -140,60 +146,83 @@ wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __re
   const int unit0 = blockIdx.x * p.upc;
   const int col_tile = blockIdx.y * dvc;       // first column of this CTA inside its heads
   const int n_blk = (p.S + TB - 1) / TB;
-  const int hw = warp - REC_CONSUMERS;
 
-  // everything token block `blk` needs, into stage `st`; an item is four tokens of one head
+  // everything token block `blk` needs, into stage `st`; an item is GPI groups of four tokens of one head
   auto prepare = [&](int blk, int st) {
-    for (int item = hw; item < p.upc * (TB / 4); item += REC_HELPERS) {
-      const int un = item / (TB / 4), grp = item % (TB / 4);
+    constexpr int ITEMS = TB / 4 / GPI;
+    const int sub = lane / LANES, c0 = (lane % LANES) * 4;
+    const unsigned mine = LANES == 32 ? 0xffffffffu : ((1u << LANES) - 1u) << (sub * LANES);
+    for (int item = warp - REC_CONSUMERS; item < p.upc * ITEMS; item += WKV_HELPERS) {
+      const int un = item / ITEMS, grp = (item % ITEMS) * GPI + (sub < GPI ? sub : 0);
       const int unit = unit0 + un, t = blk * TB + grp * 4;
-      if (unit >= units || t >= p.S) continue;
+      if (unit >= units) continue;
+      // (all lanes take part in the sums; those of a group past the end or without a group store nothing)
+      const bool stores = sub < GPI && t < p.S;
       const int b = unit / p.H, h = unit - b * p.H;
       float* base = sm + (st * p.upc + un) * unit_floats;
-      const int64_t row = (int64_t)b * p.S + t;
-      const int at = h * p.dim, c0 = lane * 4;
-      float g[CH][4][4], r[CH][4][4], k[CH][4][4], bonus[4] = {0.f, 0.f, 0.f, 0.f}, least = 1.f;
-#pragma unroll
-      for (int i = 0; i < CH; ++i) {
-        const int c = i * 128 + c0;
+      const int64_t row = (int64_t)b * p.S + (t < p.S ? t : 0);
+      const int left = p.S - t;                // tokens of this group that exist
+      const int at = h * p.dim, nv = max(0, min(dvc, p.dim - col_tile));
+      float g[CH][4][4], bonus[4] = {0.f, 0.f, 0.f, 0.f}, least = 1.f;
+      Raw4<T> r[CH][4], k[CH][4], v0[4];
+      if (p.vec) {
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
-          const int64_t rq = row + (t + q < p.S ? q : 0);
-          if (p.vec) {
-            const int cc = at + (c < p.dim ? c : 0);
+          const int64_t rq = row + (q < left ? q : 0);
+#pragma unroll
+          for (int i = 0; i < CH; ++i) {
+            const int cc = at + (i * 128 + c0 < p.dim ? i * 128 + c0 : 0);
             const float4 f = *reinterpret_cast<const float4*>(p.logits + rq * p.ld_w + cc);
             g[i][q][0] = f.x; g[i][q][1] = f.y; g[i][q][2] = f.z; g[i][q][3] = f.w;
-            load_row<T, 4>(r_in + rq * p.ld + cc, r[i][q]);
-            load_row<T, 4>(k_in + rq * p.ld + cc, k[i][q]);
-          } else {
+            r[i][q].load(r_in + rq * p.ld + cc);
+            k[i][q].load(k_in + rq * p.ld + cc);
+          }
+          v0[q].load(v_in + rq * p.ld + at + (c0 < nv ? col_tile + c0 : 0));
+        }
+      } else {
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const int64_t rq = row + (q < left ? q : 0);
+#pragma unroll
+          for (int i = 0; i < CH; ++i) {
+            float rr[4], kk[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-              const int cc = at + (c + e < p.dim ? c + e : 0);
+              const int c = i * 128 + c0 + e, cc = at + (c < p.dim ? c : 0);
               g[i][q][e] = p.logits[rq * p.ld_w + cc];
-              r[i][q][e] = rec_f<T>(r_in[rq * p.ld + cc]);
-              k[i][q][e] = rec_f<T>(k_in[rq * p.ld + cc]);
+              rr[e] = rec_f<T>(r_in[rq * p.ld + cc]);
+              kk[e] = rec_f<T>(k_in[rq * p.ld + cc]);
             }
+            r[i][q].set(rr);
+            k[i][q].set(kk);
           }
         }
       }
 #pragma unroll
-      for (int i = 0; i < CH; ++i)
+      for (int i = 0; i < CH; ++i) {
+        const int c = i * 128 + c0;
+        float w0[4], u[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int c = i * 128 + c0 + e;
-          const bool in = c < p.dim;
-          const float w0 = in ? __ldg(p.w0 + at + c) : 0.f, u = in ? __ldg(p.u + at + c) : 0.f;
-#pragma unroll
-          for (int q = 0; q < 4; ++q) {
-            const bool use = in && t + q < p.S;
-            g[i][q][e] = use ? double_exp_decay<FAST>(g[i][q][e] + w0) : 1.f;
-            if (!use) r[i][q][e] = k[i][q][e] = 0.f;
-            least = fminf(least, g[i][q][e]);
-            bonus[q] = fmaf(r[i][q][e] * u, k[i][q][e], bonus[q]);
-          }
+          w0[e] = c + e < p.dim ? __ldg(p.w0 + at + c + e) : 0.f;
+          u[e] = c + e < p.dim ? __ldg(p.u + at + c + e) : 0.f;
         }
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1)
+        for (int q = 0; q < 4; ++q) {
+          float rr[4], kk[4];
+          r[i][q].get(rr);
+          k[i][q].get(kk);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const bool use = c + e < p.dim && q < left;
+            g[i][q][e] = use ? double_exp_decay<FAST>(g[i][q][e] + w0[e]) : 1.f;
+            least = fminf(least, g[i][q][e]);
+            bonus[q] = use ? fmaf(rr[e] * u[e], kk[e], bonus[q]) : bonus[q];
+          }
+        }
+      }
+#pragma unroll
+      for (int o = LANES / 2; o > 0; o >>= 1)
 #pragma unroll
         for (int q = 0; q < 4; ++q) bonus[q] += __shfl_xor_sync(0xffffffffu, bonus[q], o);
       bool flag[4] = {false, false, false, false};
@@ -205,21 +234,25 @@ wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __re
           for (int i = 0; i < CH; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) small |= g[i][q][e] < REC_SMALL_DECAY;
-          flag[q] = __any_sync(0xffffffffu, small);
+          flag[q] = (__ballot_sync(0xffffffffu, small) & mine) != 0;
         }
       }
+      if (!stores) continue;
       // P: product of the decays since the last one that was applied directly (or the group's start)
 #pragma unroll
       for (int i = 0; i < CH; ++i) {
         const int c = i * 128 + c0;
-        if (c >= DK) continue;
         float P[4] = {1.f, 1.f, 1.f, 1.f};
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
-          float rd[4], wr[4];
+          float rr[4], kk[4];
+          r[i][q].get(rr);
+          k[i][q].get(kk);
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            rd[e] = r[i][q][e] * P[e];
+            const bool use = c + e < p.dim && q < left;
+            rr[e] = use ? rr[e] * P[e] : 0.f;
+            kk[e] = use ? kk[e] : 0.f;
             P[e] *= g[i][q][e];
           }
           if (flag[q]) {
@@ -228,23 +261,25 @@ wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __re
             for (int e = 0; e < 4; ++e) P[e] = 1.f;
           }
 #pragma unroll
-          for (int e = 0; e < 4; ++e) wr[e] = FAST ? k[i][q][e] * rcpf(P[e]) : k[i][q][e] / P[e];
-          *reinterpret_cast<float4*>(base + (grp * 4 + q) * DK + c) = make_float4(rd[0], rd[1], rd[2], rd[3]);
-          *reinterpret_cast<float4*>(base + (TB + grp * 4 + q) * DK + c) = make_float4(wr[0], wr[1], wr[2], wr[3]);
+          for (int e = 0; e < 4; ++e) kk[e] = FAST ? kk[e] * rcpf(P[e]) : kk[e] / P[e];
+          *reinterpret_cast<float4*>(base + (grp * 4 + q) * DK + c) = make_float4(rr[0], rr[1], rr[2], rr[3]);
+          *reinterpret_cast<float4*>(base + (TB + grp * 4 + q) * DK + c) = make_float4(kk[0], kk[1], kk[2], kk[3]);
         }
         *reinterpret_cast<float4*>(base + (3 * TB + grp) * DK + c) = make_float4(P[0], P[1], P[2], P[3]);
       }
       float* v = base + (3 * TB + TB / 4) * DK;
-      const int nv = max(0, min(dvc, p.dim - col_tile));
 #pragma unroll 1
-      for (int c = c0; c < dvc; c += 128) {
+      for (int c = c0; c < dvc; c += LANES * 4) {
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
           float y[4] = {0.f, 0.f, 0.f, 0.f};
-          if (t + q < p.S) {
+          if (q < left) {
             const T* src = v_in + (row + q) * p.ld + at + col_tile + c;
             if (p.vec) {
-              if (c < nv) load_row<T, 4>(src, y);
+              if (c < nv) {
+                if (c != c0) v0[q].load(src);
+                v0[q].get(y);
+              }
             } else {
 #pragma unroll
               for (int e = 0; e < 4; ++e) if (c + e < nv) y[e] = rec_f<T>(src[e]);
@@ -253,17 +288,18 @@ wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __re
           *reinterpret_cast<float4*>(v + (grp * 4 + q) * dvc + c) = make_float4(y[0], y[1], y[2], y[3]);
         }
       }
-      if (lane < 4) {
-        float* bf = v + TB * dvc;
-        bf[2 * (grp * 4 + lane)] = lane == 0 ? bonus[0] : lane == 1 ? bonus[1] : lane == 2 ? bonus[2] : bonus[3];
-        bf[2 * (grp * 4 + lane) + 1] = (lane == 0 ? flag[0] : lane == 1 ? flag[1] : lane == 2 ? flag[2] : flag[3]) ? 1.f : 0.f;
+      if (c0 == 0) {                           // bonus factors, then flags, of the group's four tokens
+        float* bf = v + TB * dvc + grp * 8;
+        *reinterpret_cast<float4*>(bf) = make_float4(bonus[0], bonus[1], bonus[2], bonus[3]);
+        *reinterpret_cast<float4*>(bf + 4) = make_float4(flag[0] ? 1.f : 0.f, flag[1] ? 1.f : 0.f, flag[2] ? 1.f : 0.f, flag[3] ? 1.f : 0.f);
       }
     }
   };
-  auto block_barrier = [] { asm volatile("bar.sync 1, %0;" ::"n"(REC_THREADS) : "memory"); };
+  auto block_barrier = [] { asm volatile("bar.sync 1, %0;" ::"n"(WKV_THREADS) : "memory"); };
 
   if (warp >= REC_CONSUMERS) {
-    asm volatile("setmaxnreg.dec.sync.aligned.u32 80;");
+    // (384 threads were launched with 168 registers each: 256 x 208 + 128 x 88 is the same sum)
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 88;");
     pdl_wait();
     pdl_trigger();
     for (int blk = 0; blk < n_blk; ++blk) {
@@ -273,7 +309,7 @@ wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __re
     block_barrier();
     return;
   }
-  asm volatile("setmaxnreg.inc.sync.aligned.u32 176;");
+  asm volatile("setmaxnreg.inc.sync.aligned.u32 208;");
   constexpr int OWN = LPC < 8 ? 8 / LPC : 1;   // columns a lane owns after a sum over its group ...
   const int j = lane % LPC, cg = lane / LPC;
   const int own = j * 8 / LPC;                 // ... starting here
@@ -295,31 +331,30 @@ wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __re
   const int b = live ? unit / p.H : 0, h = live ? unit - b * p.H : 0;
   const int64_t o_ld = (int64_t)p.H * p.dim;
   float* orow = p.o + (int64_t)b * p.S * o_ld + (int64_t)h * p.dim + col + own;
-  const bool stores = active && (LPC <= 8 || (j & (LPC / 8 - 1)) == 0);
+  int n_own = 0;                               // columns this lane stores
+  if (active && (LPC <= 8 || (j & (LPC / 8 - 1)) == 0)) n_own = max(0, min(OWN, p.dim - col - own));
   for (int blk = 0; blk < n_blk; ++blk) {
     // (all lanes of a warp belong to one head; lanes past its columns take part in the shuffles)
     if (live) {
       const float* base = sm + ((blk & 1) * p.upc + un) * unit_floats;
       const float* vb = base + (3 * TB + TB / 4) * DK + lcol;
-      const float* bf = base + (3 * TB + TB / 4) * DK + TB * dvc;
       const int t0 = blk * TB, n = min(TB, p.S - t0);
-      auto token = [&](int t, float (&po)[8]) {
+      auto read = [&](int t, float (&po)[8]) {
         const float4* r4 = reinterpret_cast<const float4*>(base + t * DK) + j;
-        const float4* k4 = reinterpret_cast<const float4*>(base + (TB + t) * DK) + j;
         float2 acc[8];
-#pragma unroll
-        for (int c = 0; c < 8; ++c) acc[c] = make_float2(0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const float4 r = r4[i * LPC];
 #pragma unroll
-          for (int c = 0; c < 8; ++c) acc[c] = fma2(s[c][2 * i], make_float2(r.x, r.y), acc[c]);
+          for (int c = 0; c < 8; ++c) acc[c] = i ? fma2(s[c][2 * i], make_float2(r.x, r.y), acc[c]) : mul2(s[c][0], make_float2(r.x, r.y));
 #pragma unroll
           for (int c = 0; c < 8; ++c) acc[c] = fma2(s[c][2 * i + 1], make_float2(r.z, r.w), acc[c]);
         }
 #pragma unroll
         for (int c = 0; c < 8; ++c) po[c] = acc[c].x + acc[c].y;
-        if (bf[2 * t + 1] != 0.f) state_scale<LPC>(s, reinterpret_cast<const float4*>(base + (2 * TB + t) * DK) + j);
+      };
+      auto write = [&](int t) {
+        const float4* k4 = reinterpret_cast<const float4*>(base + (TB + t) * DK) + j;
         const float4 va = *reinterpret_cast<const float4*>(vb + t * dvc), vc = *reinterpret_cast<const float4*>(vb + t * dvc + 4);
         const float v[8] = {va.x, va.y, va.z, va.w, vc.x, vc.y, vc.z, vc.w};
 #pragma unroll
@@ -331,23 +366,46 @@ wkv_kernel(const T* __restrict__ r_in, const T* __restrict__ k_in, const T* __re
           for (int c = 0; c < 8; ++c) s[c][2 * i + 1] = fma2(make_float2(k.z, k.w), make_float2(v[c], v[c]), s[c][2 * i + 1]);
         }
       };
-      auto finish = [&](int t, const float (&po)[8]) {
-        if (!stores || t >= n) return;
+      auto finish = [&](int t, float bonus, const float (&po)[8]) {
         float* ot = orow + (int64_t)(t0 + t) * o_ld;
 #pragma unroll
         for (int i = 0; i < OWN; ++i)
-          if (col + own + i < p.dim) ot[i] = fmaf(bf[2 * t], vb[t * dvc + own + i], po[i]);
+          if (i < n_own && t < n) ot[i] = fmaf(bonus, vb[t * dvc + own + i], po[i]);
       };
       // (tokens past the end of a group of four hold zeros and decays of one)
 #pragma unroll 1
-      for (int t = 0; t < n; t += 2) {
+      for (int t = 0; t < n; t += 4) {
+        const float* bf = base + (3 * TB + TB / 4) * DK + TB * dvc + t * 2;
+        const float4 bonus = *reinterpret_cast<const float4*>(bf), flag = *reinterpret_cast<const float4*>(bf + 4);
         float pa[8], pb[8];
-        token(t, pa);
-        token(t + 1, pb);
-        group_sums<LPC>(j, pa, pb);
-        finish(t, pa);
-        finish(t + 1, pb);
-        if ((t & 3) == 2 || t + 2 >= n) state_scale<LPC>(s, reinterpret_cast<const float4*>(base + (3 * TB + (t >> 2)) * DK) + j);
+        if (flag.x + flag.y + flag.z + flag.w == 0.f) {
+          read(t, pa);
+          write(t);
+          read(t + 1, pb);
+          write(t + 1);
+          group_sums<LPC>(j, pa, pb);
+          finish(t, bonus.x, pa);
+          finish(t + 1, bonus.y, pb);
+          read(t + 2, pa);
+          write(t + 2);
+          read(t + 3, pb);
+          write(t + 3);
+          group_sums<LPC>(j, pa, pb);
+          finish(t + 2, bonus.z, pa);
+          finish(t + 3, bonus.w, pb);
+        } else {
+#pragma unroll 1
+          for (int q = 0; q < 4; ++q) {
+            read(t + q, pa);
+            if (bf[4 + q] != 0.f) state_scale<LPC>(s, reinterpret_cast<const float4*>(base + (2 * TB + t + q) * DK) + j);
+            write(t + q);
+#pragma unroll
+            for (int c = 0; c < 8; ++c) pb[c] = 0.f;
+            group_sums<LPC>(j, pa, pb);
+            finish(t + q, bf[q], pa);
+          }
+        }
+        state_scale<LPC>(s, reinterpret_cast<const float4*>(base + (3 * TB + (t >> 2)) * DK) + j);
       }
     }
     block_barrier();
@@ -441,7 +499,7 @@ static int launch_wkv(const void* r, const void* k, const void* v, WkvParams p) 
     configured[ctx().device & 63] = true;
   }
   dim3 grid((units + p.upc - 1) / p.upc, col_tiles);
-  KD_CUDA_CHECK(launch_ex(wkv_kernel<T, LPC>, grid, dim3(REC_THREADS), (size_t)smem, (const T*)r, (const T*)k, (const T*)v, p));
+  KD_CUDA_CHECK(launch_ex(wkv_kernel<T, LPC>, grid, dim3(WKV_THREADS), (size_t)smem, (const T*)r, (const T*)k, (const T*)v, p));
   return after_launch("wkv_kernel");
 }
 
