@@ -607,13 +607,49 @@ struct DeltaOutParams {
   int w_head;                   // norm weights: stride from one head's to the next (0: shared by the heads)
 };
 
-template <typename T>
+// LPH lanes a head (vdim = 4 LPH), 32 / LPH heads a warp; LPH = 0: any size, one head a warp.
+template <typename T, int LPH>
 __global__ void __launch_bounds__(256)
 delta_out_kernel(const float* __restrict__ o, const T* __restrict__ gate, const float* __restrict__ w, const T* __restrict__ proj,
                  T* __restrict__ hist, T* __restrict__ out, DeltaOutParams p) {
   pdl_wait();
   pdl_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (LPH > 0 && (int)blockIdx.x < p.out_blocks) {
+    constexpr int HEADS = LPH > 0 ? 32 / (LPH > 0 ? LPH : 1) : 1;
+    const int64_t items = (int64_t)p.B * p.S * p.H, own = ((int64_t)blockIdx.x * 8 + warp) * HEADS + lane / (LPH > 0 ? LPH : 1);
+    const int64_t item = own < items ? own : items - 1;      // (lanes without a head join the sums)
+    const int64_t t = item / p.H;
+    const int h = (int)(item - t * p.H), c = (lane % (LPH > 0 ? LPH : 1)) * 4;
+    const float4 x = *reinterpret_cast<const float4*>(o + item * p.vdim + c);
+    Raw4<T> graw;
+    graw.load(gate + t * p.ld_gate + h * p.vdim + c);
+    const float4 wv = *reinterpret_cast<const float4*>(w + h * p.w_head + c);
+    float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
+#pragma unroll
+    for (int k = LPH / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+    if (own >= items) return;
+    const float inv = 1.0f / sqrtf(ss / (float)p.vdim + p.eps);
+    float z[4];
+    graw.get(z);
+    const float xs[4] = {x.x, x.y, x.z, x.w}, ws[4] = {wv.x, wv.y, wv.z, wv.w};
+    float y[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float g = rec_sigmoid<sizeof(T) == 2>(z[e]);
+      y[e] = xs[e] * inv * ws[e] * (p.gate_silu ? z[e] * g : g);
+    }
+    if constexpr (sizeof(T) == 2) {
+      __nv_bfloat162 a = __floats2bfloat162_rn(y[0], y[1]), b = __floats2bfloat162_rn(y[2], y[3]);
+      uint2 u;
+      u.x = *reinterpret_cast<uint32_t*>(&a);
+      u.y = *reinterpret_cast<uint32_t*>(&b);
+      *reinterpret_cast<uint2*>(out + item * p.vdim + c) = u;
+    } else {
+      *reinterpret_cast<float4*>(out + item * p.vdim + c) = make_float4(y[0], y[1], y[2], y[3]);
+    }
+    return;
+  }
   if ((int)blockIdx.x < p.out_blocks) {
     const int64_t item = (int64_t)blockIdx.x * 8 + warp;
     if (item >= (int64_t)p.B * p.S * p.H) return;
@@ -641,6 +677,19 @@ delta_out_kernel(const float* __restrict__ o, const T* __restrict__ gate, const 
     const int t = p.S - halo + r;
     hb[(int64_t)r * p.hist_ld] = t >= 0 ? proj[((int64_t)b * p.S + t) * p.ld + p.conv_col + ch] : hb[(int64_t)(t + halo) * p.hist_ld];
   }
+}
+
+template <typename T>
+static int launch_delta_out(const float* o, const T* gate, const float* w, const T* proj, T* hist, T* out, DeltaOutParams p) {
+  const bool vec = p.ld_gate % 4 == 0 && p.w_head % 4 == 0 && reinterpret_cast<uintptr_t>(gate) % (4 * sizeof(T)) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const int lph = vec && (p.vdim == 16 || p.vdim == 32 || p.vdim == 64 || p.vdim == 128) ? p.vdim / 4 : 0;
+  const int64_t per = lph ? 8 * (32 / lph) : 8;
+  p.out_blocks = (int)(((int64_t)p.B * p.S * p.H + per - 1) / per);
+  const int hist_blocks = p.taps > 1 ? (int)(((int64_t)p.B * p.channels + 255) / 256) : 0;
+  auto k = lph == 4 ? delta_out_kernel<T, 4> : lph == 8 ? delta_out_kernel<T, 8> : lph == 16 ? delta_out_kernel<T, 16> : lph == 32 ? delta_out_kernel<T, 32> : delta_out_kernel<T, 0>;
+  KD_CUDA_CHECK(launch_ex(k, dim3(p.out_blocks + hist_blocks), dim3(256), 0, o, gate, w, proj, hist, out, p));
+  return after_launch("delta_out_kernel");
 }
 
 static int f32_vec(const kd_tensor* t, int64_t n, const char* what, const float** out) {
@@ -785,20 +834,15 @@ KD_API int kd_delta_out(const kd_tensor* o, const kd_tensor* gate, const kd_tens
   p.eps = eps;
   KD_REQUIRE(gate_act == KD_GATE_SIGMOID || gate_act == KD_GATE_SILU, "unknown gate activation %d", gate_act);
   p.gate_silu = gate_act == KD_GATE_SILU;
-  p.out_blocks = (int)((T * p.H + 7) / 8);
-  const int hist_blocks = taps > 1 ? (int)(((int64_t)p.B * p.channels + 255) / 256) : 0;
   void *po, *pg, *pp, *ph, *pout;
   KD_TRY(tensor_ptr(o, &po));
   KD_TRY(tensor_ptr(gate, &pg));
   KD_TRY(tensor_ptr(proj, &pp));
   KD_TRY(tensor_ptr(history, &ph));
   KD_TRY(tensor_ptr(out, &pout));
-  dim3 grid(p.out_blocks + hist_blocks);
   if (proj->dtype == KD_BF16)
-    KD_CUDA_CHECK(launch_ex(delta_out_kernel<__nv_bfloat16>, grid, dim3(256), 0, (const float*)po, (const __nv_bfloat16*)pg, w, (const __nv_bfloat16*)pp, (__nv_bfloat16*)ph, (__nv_bfloat16*)pout, p));
-  else
-    KD_CUDA_CHECK(launch_ex(delta_out_kernel<float>, grid, dim3(256), 0, (const float*)po, (const float*)pg, w, (const float*)pp, (float*)ph, (float*)pout, p));
-  return after_launch("delta_out_kernel");
+    return launch_delta_out<__nv_bfloat16>((const float*)po, (const __nv_bfloat16*)pg, w, (const __nv_bfloat16*)pp, (__nv_bfloat16*)ph, (__nv_bfloat16*)pout, p);
+  return launch_delta_out<float>((const float*)po, (const float*)pg, w, (const float*)pp, (float*)ph, (float*)pout, p);
 }
 
 KD_API int kd_gated_head_norm(const kd_tensor* o, const kd_tensor* gate, const kd_tensor* norm_weight, int heads, float eps, int gate_act,
@@ -819,14 +863,11 @@ KD_API int kd_gated_head_norm(const kd_tensor* o, const kd_tensor* gate, const k
   KD_REQUIRE(out->dtype == gate->dtype && is_contiguous(out) && numel(out) == numel(o), "out must be [T, heads*vdim] of gate's type");
   if (T == 0) return KD_OK;
   p.ld_gate = gate->strides[0];
-  p.out_blocks = (int)((T * p.H + 7) / 8);
   void *po, *pg, *pout;
   KD_TRY(tensor_ptr(o, &po));
   KD_TRY(tensor_ptr(gate, &pg));
   KD_TRY(tensor_ptr(out, &pout));
   if (gate->dtype == KD_BF16)
-    KD_CUDA_CHECK(launch_ex(delta_out_kernel<__nv_bfloat16>, dim3(p.out_blocks), dim3(256), 0, (const float*)po, (const __nv_bfloat16*)pg, w, (const __nv_bfloat16*)nullptr, (__nv_bfloat16*)nullptr, (__nv_bfloat16*)pout, p));
-  else
-    KD_CUDA_CHECK(launch_ex(delta_out_kernel<float>, dim3(p.out_blocks), dim3(256), 0, (const float*)po, (const float*)pg, w, (const float*)nullptr, (float*)nullptr, (float*)pout, p));
-  return after_launch("delta_out_kernel");
+    return launch_delta_out<__nv_bfloat16>((const float*)po, (const __nv_bfloat16*)pg, w, nullptr, nullptr, (__nv_bfloat16*)pout, p);
+  return launch_delta_out<float>((const float*)po, (const float*)pg, w, nullptr, nullptr, (float*)pout, p);
 }

@@ -745,6 +745,7 @@ struct SkinnyParams {
   float* tail;            // weight rows from tail_row on: fp32 [Mb][ld_tail] instead of the bf16 output
   int tail_row, ld_tail;
   float alpha;            // factor of the fp32 outputs
+  int group_tiles;        // weight tiles per group: group g holds W rows [g N, (g+1) N), x and output rows [g Mb, (g+1) Mb)
   int* err;
 };
 
@@ -763,7 +764,7 @@ gemm_skinny_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n_tile = blockIdx.x, split = blockIdx.y;
+  const int group = blockIdx.x / p.group_tiles, n_tile = blockIdx.x - group * p.group_tiles, split = blockIdx.y;
   const int total_kb = (p.K + GEMM_BK - 1) / GEMM_BK;
   const int kb_begin = split * p.kblocks_per_split;
   const int kb_end = min(total_kb, kb_begin + p.kblocks_per_split);
@@ -796,8 +797,8 @@ gemm_skinny_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
         if (!mbar_wait(&empty[stage], phase ^ 1, abort_flag, p.err, 211)) break;
         uint8_t* sw = smem + stage * stage_bytes;
         mbar_arrive_expect_tx(&full[stage], (uint32_t)stage_bytes);
-        tma_load_2d(sw, &tmap_w, &full[stage], (kb_begin + i) * GEMM_BK, n_tile * 128);
-        tma_load_2d(sw + W_BYTES, &tmap_x, &full[stage], (kb_begin + i) * GEMM_BK, 0);
+        tma_load_2d(sw, &tmap_w, &full[stage], (kb_begin + i) * GEMM_BK, group * p.N + n_tile * 128);
+        tma_load_2d(sw + W_BYTES, &tmap_x, &full[stage], (kb_begin + i) * GEMM_BK, group * p.Mb);
         if (++stage == p.stages) { stage = 0; phase ^= 1; }
       }
     }
@@ -859,7 +860,7 @@ gemm_skinny_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
             const int m = c0 + i;
             if (m < p.Mb) {
               if (p.tail && n >= p.tail_row) p.tail[(int64_t)m * p.ld_tail + (n - p.tail_row)] = __uint_as_float(r[i]);
-              else if (p.out_bf16) p.out_bf16[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(__uint_as_float(r[i]));
+              else if (p.out_bf16) p.out_bf16[(int64_t)(group * p.Mb + m) * p.ldo + n] = __float2bfloat16_rn(__uint_as_float(r[i]));
               else p.out_f32[((int64_t)split * p.Mb + m) * p.N + n] = __uint_as_float(r[i]) * p.alpha;
             }
           }
@@ -891,11 +892,12 @@ int gemm_skinny_auto_splits(int N, int K) {
 // x [Mb<=128, K] bf16, W [N, K] bf16 -> fp32 partials [splits][Mb][N] (or bf16 [Mb][N] when
 // out_bf16 != NULL and splits == 1).
 int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int Mb, int N, int K, int splits,
-                     float* out_f32, void* out_bf16, int glu, float alpha, float* tail, int tail_row, int ld_tail) {
+                     float* out_f32, void* out_bf16, int glu, float alpha, float* tail, int tail_row, int ld_tail, int groups) {
   KD_REQUIRE(Mb >= 1 && Mb <= 128, "skinny gemm: %d rows; this path handles 1..128", Mb);
   KD_REQUIRE(N > 0 && K > 0 && K % 8 == 0, "skinny gemm: K=%d must be a positive multiple of 8", K);
   KD_REQUIRE(splits >= 1, "skinny gemm: splits must be >= 1");
   KD_REQUIRE(out_bf16 == nullptr || splits == 1, "skinny gemm: bf16 output needs splits == 1");
+  KD_REQUIRE(groups >= 1 && (groups == 1 || (out_bf16 != nullptr && !glu && !tail)), "skinny gemm: groups need the plain bf16 output");
   KD_REQUIRE(!glu || (out_bf16 != nullptr && N % 32 == 0), "skinny gemm: the gated epilogue needs a bf16 output and N %% 32 == 0");
   SkinnyParams p{};
   p.Mb = Mb; p.N = N; p.K = K;
@@ -911,7 +913,7 @@ int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int
   if (stages > p.kblocks_per_split) stages = p.kblocks_per_split < 2 ? 2 : p.kblocks_per_split;
   // many tiles (lm_head): a shallower ring lets two CTAs share an SM, so that one CTA's prologue and
   // epilogue overlap the other's streaming
-  if ((int64_t)((N + 127) / 128) * splits >= 2 * ctx().sm_count) {
+  if ((int64_t)((N + 127) / 128) * splits * groups >= 2 * ctx().sm_count) {
     const int two_per_sm = (108 * 1024) / stage_bytes;
     if (stages > two_per_sm) stages = two_per_sm;
   }
@@ -923,17 +925,18 @@ int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int
   p.alpha = alpha;
   p.tail = tail; p.tail_row = tail_row; p.ld_tail = ld_tail;
   p.ldo = tail ? tail_row : N;
+  p.group_tiles = (N + 127) / 128;
   p.err = ctx().error_flag;
   CUtensorMap tw, tx;
-  KD_TRY(make_tmap_bf16_2d(&tw, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, 128, GEMM_BK));
-  KD_TRY(make_tmap_bf16_2d(&tx, x, (uint64_t)Mb, (uint64_t)K, (uint64_t)ldx, (uint32_t)p.x_box, GEMM_BK));
+  KD_TRY(make_tmap_bf16_2d(&tw, W, (uint64_t)N * groups, (uint64_t)K, (uint64_t)ldw, 128, GEMM_BK));
+  KD_TRY(make_tmap_bf16_2d(&tx, x, (uint64_t)Mb * groups, (uint64_t)K, (uint64_t)ldx, (uint32_t)p.x_box, GEMM_BK));
   const int smem = stages * stage_bytes + 1024 + 256;
   static bool skinny_configured[64] = {false};   // per device
   if (!skinny_configured[ctx().device & 63]) {
     KD_CUDA_CHECK(cudaFuncSetAttribute(gemm_skinny_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 210 * 1024));
     skinny_configured[ctx().device & 63] = true;
   }
-  dim3 grid((N + 127) / 128, splits);
+  dim3 grid(p.group_tiles * groups, splits);
   KD_CUDA_CHECK(launch_ex(gemm_skinny_tcgen05_kernel, grid, dim3(GEMM_THREADS), (size_t)smem, tw, tx, p));
   return after_launch("gemm_skinny_tcgen05_kernel");
 }

@@ -40,10 +40,11 @@ int gemm_bf16_qkv_rope(const void* A, int64_t lda, const void* W, int64_t ldw, i
                        void* k_cache, void* v_cache, int64_t kc_b, int64_t kc_h, int64_t kc_s);
 int gemm_skinny_auto_splits(int N, int K);
 // x [Mb<=128,K] * W[N,K]^T -> fp32 partials [splits][Mb][N], or bf16 [Mb][N] when out_bf16 != NULL (splits == 1).
+// groups > 1: as many independent problems, x [groups][Mb][K], W [groups][N][K], bf16 out [groups][Mb][N].
 // glu (bf16 output [Mb][N/2], interleaved rows): 0 none, 1 silu(gate) * up, 2 gelu(gate) * up.
 int gemm_bf16_skinny(const void* x, int64_t ldx, const void* W, int64_t ldw, int Mb, int N, int K, int splits,
                      float* out_f32, void* out_bf16, int glu, float alpha = 1.0f, float* tail = nullptr, int tail_row = 0,
-                     int ld_tail = 0);
+                     int ld_tail = 0, int groups = 1);
 size_t attention_decode_scratch_bytes(int B, int Hkv, int group, int splits, int D);
 int attention_decode(const kd_tensor* q, const kd_tensor* k, const kd_tensor* v, const kd_tensor* out, float scale,
                      const int* ctx_dev, int ctx_host, const int* block_table, int max_pages, int splits,

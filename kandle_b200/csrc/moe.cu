@@ -251,8 +251,12 @@ static void launch_moe_linear(const void* x, const void* w, const int* off, int 
 static int grouped_linear(int dtype, const void* x, const void* w, const int* off, int64_t R, int64_t E, int64_t N, int64_t K, int epi, float limit, void* out) {
   const int64_t n_out = epi != KD_EPI_NONE ? N / 2 : N;
   if (dtype == KD_BF16 && K % 8 == 0 && n_out % 8 == 0 && epi != KD_EPI_SWIGLU &&
-      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0)
+      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+    // equal groups of a few rows: stream the weights, where the 128-row weight tiles are enough to fill the GPU
+    if (!off && epi == KD_EPI_NONE && R / E <= 64 && E * ((N + 127) / 128) >= ctx().sm_count / 2)
+      return gemm_bf16_skinny(x, K, w, K, (int)(R / E), (int)N, (int)K, 1, nullptr, out, 0, 1.0f, nullptr, 0, 0, (int)E);
     return gemm_bf16_grouped(x, w, out, off, (int)R, (int)E, (int)N, (int)K, epi, limit);
+  }
   const int64_t tiles = R / GL_BM + (E < R ? E : R) + 1;
   KD_REQUIRE(tiles <= 65535, "grouped linear (CUDA cores): too many row tiles (%lld)", (long long)tiles);
   dim3 grid((unsigned)((n_out + GL_BN - 1) / GL_BN), (unsigned)tiles);

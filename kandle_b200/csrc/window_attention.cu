@@ -42,12 +42,14 @@ __device__ __forceinline__ uint32_t wa_pack(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+constexpr int QK_THREADS = 128;     // small CTAs: a token is a chain of latencies, so many of them share an SM
+
 // One CTA a token; the query and key rows pass through shared memory as fp32.
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(QK_THREADS, 8)
 qk_prep_kernel(const T* __restrict__ proj, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, QkPrepParams p) {
   extern __shared__ __align__(16) float row_s[];      // [(H + G) * dim] weighted values before the scale
-  __shared__ float red[2][8];
+  __shared__ float red[2][QK_THREADS / 32];
   pdl_wait();
   pdl_trigger();
   const int64_t token = blockIdx.x;
@@ -61,7 +63,7 @@ qk_prep_kernel(const T* __restrict__ proj, T* __restrict__ q_out, T* __restrict_
   const int nq = p.H * p.dim, nk = p.k_col >= 0 ? p.G * p.dim : 0, tid = threadIdx.x;
   float sq = 0.f, sk = 0.f;
   if (sizeof(T) == 2 && p.vec) {
-    for (int i = tid * 8; i < nq + nk; i += 256 * 8) {
+    for (int i = tid * 8; i < nq + nk; i += QK_THREADS * 8) {
       const bool is_q = i < nq;
       const uint4 u = *reinterpret_cast<const uint4*>(row + (is_q ? p.q_col + i : p.k_col + i - nq));
       const float* w = is_q ? p.qw + i : p.kw + i - nq;
@@ -76,7 +78,7 @@ qk_prep_kernel(const T* __restrict__ proj, T* __restrict__ q_out, T* __restrict_
       *reinterpret_cast<float4*>(row_s + i + 4) = make_float4(v[4] * w1.x, v[5] * w1.y, v[6] * w1.z, v[7] * w1.w);
     }
   } else {
-    for (int i = tid; i < nq + nk; i += 256) {
+    for (int i = tid; i < nq + nk; i += QK_THREADS) {
       const bool is_q = i < nq;
       const float v = wa_f<T>(row[is_q ? p.q_col + i : p.k_col + i - nq]);
       if (is_q) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
@@ -89,7 +91,7 @@ qk_prep_kernel(const T* __restrict__ proj, T* __restrict__ q_out, T* __restrict_
   __syncthreads();
   sq = sk = 0.f;
 #pragma unroll
-  for (int w = 0; w < 8; ++w) { sq += red[0][w]; sk += red[1][w]; }
+  for (int w = 0; w < QK_THREADS / 32; ++w) { sq += red[0][w]; sk += red[1][w]; }
   const float iq = 1.0f / sqrtf(sq / (float)nq + p.eps), ik = nk ? 1.0f / sqrtf(sk / (float)nk + p.eps) : 0.f;
   const int n2 = p.rot / 2;
   const float* cs = p.cos_t + (int64_t)pos * n2;
@@ -109,7 +111,7 @@ qk_prep_kernel(const T* __restrict__ proj, T* __restrict__ q_out, T* __restrict_
   };
   if (sizeof(T) == 2 && p.vec) {
     const int pieces = p.dq / 8;
-    for (int i = tid; i < heads * pieces; i += 256) {
+    for (int i = tid; i < heads * pieces; i += QK_THREADS) {
       const int x = i / pieces, e = (i - x * pieces) * 8;
       float y[8];
       if (p.rot % 16 == 0 && e < p.dim) {       // eight entries lie on one side of every boundary
@@ -144,19 +146,19 @@ qk_prep_kernel(const T* __restrict__ proj, T* __restrict__ q_out, T* __restrict_
     }
     if (!nk) return;
     const int vp = p.dv / 8;
-    for (int i = tid; i < p.G * vp; i += 256) {
+    for (int i = tid; i < p.G * vp; i += QK_THREADS) {
       const int x = i / vp, e = (i - x * vp) * 8;
       const uint4 u = e < p.vdim ? *reinterpret_cast<const uint4*>(row + p.v_col + x * p.vdim + e) : make_uint4(0, 0, 0, 0);
       *reinterpret_cast<uint4*>(v_cache + (int64_t)b * p.vc_b + (int64_t)x * p.vc_h + (int64_t)pos * p.vc_s + e) = u;
     }
     return;
   }
-  for (int i = tid; i < heads * p.dq; i += 256) {
+  for (int i = tid; i < heads * p.dq; i += QK_THREADS) {
     const int x = i / p.dq, e = i - x * p.dq;
     dest(x)[e] = wa_t<T>(entry(x, e));
   }
   if (!nk) return;
-  for (int i = tid; i < p.G * p.dv; i += 256) {
+  for (int i = tid; i < p.G * p.dv; i += QK_THREADS) {
     const int x = i / p.dv, e = i - x * p.dv;
     v_cache[(int64_t)b * p.vc_b + (int64_t)x * p.vc_h + (int64_t)pos * p.vc_s + e] = e < p.vdim ? row[p.v_col + x * p.vdim + e] : wa_t<T>(0.f);
   }
@@ -363,9 +365,9 @@ KD_API int kd_qk_norm_rope_cache(const kd_tensor* proj, int q_col, int k_col, in
     configured[ctx().device & 63] = true;
   }
   if (proj->dtype == KD_BF16)
-    KD_CUDA_CHECK(launch_ex(qk_prep_kernel<__nv_bfloat16>, dim3((unsigned)tokens), dim3(256), smem, (const __nv_bfloat16*)pp, (__nv_bfloat16*)pq, (__nv_bfloat16*)pk, (__nv_bfloat16*)pv, p));
+    KD_CUDA_CHECK(launch_ex(qk_prep_kernel<__nv_bfloat16>, dim3((unsigned)tokens), dim3(QK_THREADS), smem, (const __nv_bfloat16*)pp, (__nv_bfloat16*)pq, (__nv_bfloat16*)pk, (__nv_bfloat16*)pv, p));
   else
-    KD_CUDA_CHECK(launch_ex(qk_prep_kernel<float>, dim3((unsigned)tokens), dim3(256), smem, (const float*)pp, (float*)pq, (float*)pk, (float*)pv, p));
+    KD_CUDA_CHECK(launch_ex(qk_prep_kernel<float>, dim3((unsigned)tokens), dim3(QK_THREADS), smem, (const float*)pp, (float*)pq, (float*)pk, (float*)pv, p));
   return after_launch("qk_prep_kernel");
 }
 
