@@ -48,6 +48,7 @@ constexpr float REC_LOG2E = 1.4426950408889634f;
 template <bool FAST> __device__ __forceinline__ float rec_sigmoid(float x) {
   return FAST ? rcpf(1.0f + ex2f(-REC_LOG2E * x)) : 1.0f / (1.0f + expf(-x));
 }
+
 // Four consecutive channels of a row as they lie in memory.
 template <typename T> struct Raw4;
 template <> struct Raw4<__nv_bfloat16> {
